@@ -99,13 +99,14 @@ SYMBOLS += [
 class CRotarySpec(ctypes.Structure):
     """``cake_b200_rotary_spec`` (include/cake_b200.h)."""
     _fields_ = [("dims", c_int), ("base", ctypes.c_double), ("yarn_factor", ctypes.c_double), ("yarn_fast", ctypes.c_double),
-                ("yarn_slow", ctypes.c_double), ("yarn_original", c_int)]
+                ("yarn_slow", ctypes.c_double), ("yarn_original", c_int), ("interleaved", c_int), ("stretch_factor", ctypes.c_double),
+                ("stretch_low", ctypes.c_double), ("stretch_high", ctypes.c_double), ("stretch_original", ctypes.c_double)]
 
 
 class CMoeSpec(ctypes.Structure):
     """``cake_b200_moe_spec`` (include/cake_b200.h)."""
     _fields_ = [("experts", c_int), ("identity", c_int), ("top", c_int), ("scale", c_float), ("ff", c_int), ("shared_ff", c_int), ("act", c_int),
-                ("limit", c_float), ("shared_limit", c_float), ("logit_bias", c_int)]
+                ("limit", c_float), ("shared_limit", c_float), ("logit_bias", c_int), ("groups", c_int), ("groups_keep", c_int), ("plain_weights", c_int)]
 
 
 class CMixerSpec(ctypes.Structure):
@@ -118,7 +119,8 @@ CMixerSpec._fields_ = [("kind", c_int), ("heads", c_int), ("dim", c_int), ("vdim
                        ("kv_heads", c_int), ("bias_rows", c_int), ("bias_max", c_float), ("gate_cap", c_float), ("norm_offset", c_float),
                        ("canon_taps", c_int), ("dense_ff", c_int), ("dense_act", c_int), ("dense_limit", c_float), ("side", POINTER(CMixerSpec)),
                        ("window", c_int), ("keep_first", c_int), ("qk_unit", c_int), ("q_rank", c_int), ("norm_kind", c_int), ("norm_alpha", c_float * 4),
-                       ("side_dim", c_int), ("side_col", c_int)]
+                       ("side_dim", c_int), ("side_col", c_int), ("pool", c_int), ("chunk", c_int), ("softcap", c_float), ("sink_zero", c_int),
+                       ("qk_norm", c_int), ("v_unit", c_int), ("branch_scale", c_float)]
 
 
 MIXER_TENSOR_FIELDS = ("norm1", "norm2", "q", "k", "v", "g", "o", "dkv", "dkv_norm", "uk", "uv", "in", "conv", "conv_b", "dt_bias", "a_log", "d",
@@ -133,7 +135,8 @@ class CMixerTensors(ctypes.Structure):
 
 
 # fields behind `side` in the C struct (the newer mechanisms)
-MIXER_TENSOR_FIELDS_2 = ("sink", "dq", "dq_norm", "uq", "norm1_b", "post1_b", "norm2_b", "post2_b", "side_gate", "side_proj", "side_norm")
+MIXER_TENSOR_FIELDS_2 = ("sink", "dq", "dq_norm", "uq", "norm1_b", "post1_b", "norm2_b", "post2_b", "side_gate", "side_proj", "side_norm",
+                         "q_norm", "k_norm")
 CMixerTensors._fields_ = [(n, POINTER(_VP) if n.startswith("e_") else _VP) for n in MIXER_TENSOR_FIELDS] + [("side", POINTER(CMixerTensors))] + \
                          [(n, _VP) for n in MIXER_TENSOR_FIELDS_2]
 
@@ -142,7 +145,7 @@ class CEmbedTables(ctypes.Structure):
     """``cake_b200_embed_tables`` (include/cake_b200.h)."""
     _fields_ = [("bigram", _VP), ("bigram_rows", c_int), ("mul_prev", c_int), ("mul_cur", c_int), ("pos", _VP), ("pos_rows", c_int),
                 ("final_norm_offset", c_float), ("side", _VP), ("side_cols", c_int), ("final_norm_kind", c_int), ("final_alpha", c_float),
-                ("final_bias", _VP)]
+                ("final_bias", _VP), ("embed_norm", _VP)]
 
 
 SYMBOLS += [

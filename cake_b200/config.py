@@ -48,13 +48,29 @@ class LayerSpec:
 @dataclass
 class RotarySpec:
     """``cake_b200_rotary_spec``: rotation of the first ``dims`` entries of a head, pair (i, i + dims/2); ``factor`` > 0 blends
-    the frequencies towards f / factor between the pairs that complete ``fast`` and ``slow`` turns over ``original`` positions."""
+    the frequencies towards f / factor between the pairs that complete ``fast`` and ``slow`` turns over ``original`` positions.
+    ``interleaved``: pairs (2i, 2i + 1).  ``stretch`` = (factor, low, high, original): wavelengths above original / low are stretched
+    by ``factor``, those below original / high are kept, the ones between are interpolated."""
     dims: int = 0
     base: float = 10000.0
     factor: float = 0.0
     fast: float = 0.0
     slow: float = 0.0
     original: int = 0
+    interleaved: bool = False
+    stretch: tuple = ()
+
+    @staticmethod
+    def stretched(d: Optional[dict], interleaved: bool) -> "RotarySpec":
+        """``rot`` = {dims, base, scaling: {factor, low, high, original} or absent} with the stretched-wavelength scaling."""
+        if not d or not int(d.get("dims") or 0):
+            return RotarySpec(interleaved=interleaved)
+        sc = d.get("scaling")
+        r = RotarySpec(dims=int(d["dims"]), base=float(d["base"]), interleaved=interleaved,
+                       stretch=tuple(float(sc[k]) for k in ("factor", "low", "high", "original")) if sc else ())
+        if r.dims % 2 or not r.base > 0 or (r.stretch and not (r.stretch[0] > 0 and 0 < r.stretch[1] < r.stretch[2] and r.stretch[3] > 0)):
+            raise ValueError(f"bad rotation {d}")
+        return r
 
     @staticmethod
     def from_dict(d: Optional[dict]) -> "RotarySpec":
@@ -68,6 +84,8 @@ class RotarySpec:
         if not self.dims:
             return None
         d = {"dims": self.dims, "base": self.base}
+        if self.stretch:
+            d["scaling"] = dict(zip(("factor", "low", "high", "original"), self.stretch))
         if self.factor:
             d["scaling"] = {"factor": self.factor, "fast": self.fast, "slow": self.slow, "original": self.original}
         return d
@@ -83,10 +101,13 @@ class MoeSpec:
     scale: float = 1.0
     ff: int = 0
     shared_ff: int = 0
-    act: int = 0             # 0 silu, 1 tanh-gelu, 2 clamped (min(g, limit) sigmoid(1.702 g) (clamp(u) + 1))
+    act: int = 0             # 0 silu, 1 tanh-gelu, 2 clamped (min(g, limit) sigmoid(1.702 g) (clamp(u) + 1)), 3 relu
     limit: float = 0.0
     shared_limit: float = 0.0
     logit_bias: bool = False  # the router's correction is a bias of the logits; choice by logit, softmax over the chosen alone
+    groups: int = 0          # > 1: equal groups of neighbouring experts; only those of the ``groups_keep`` groups with the best score may be chosen
+    groups_keep: int = 0
+    plain_weights: bool = False  # the weights are the chosen experts' scores, not renormalised
 
 
 MIXER_KINDS = {"latent_attention": 1, "retention": 2, "mamba2": 3, "delta": 4, "talking_attention": 5, "matrix_memory": 6,
@@ -122,7 +143,7 @@ class MixerSpec:
     post_norms: bool = False
     canon_taps: int = 0
     dense_ff: int = 0
-    dense_act: int = 0       # 0 silu, 1 tanh-gelu, 2 clamped (min(g, limit) sigmoid(1.702 g) (clamp(u) + 1))
+    dense_act: int = 0       # 0 silu, 1 tanh-gelu, 2 clamped (min(g, limit) sigmoid(1.702 g) (clamp(u) + 1)), 3 relu
     dense_limit: float = 0.0
     side: Optional["MixerSpec"] = None   # a second mixer beside this one, reading the same input
     # sink_attention (grouped-query attention with a rotation of part of every head, unit-RMS q and k, a sliding window that keeps
@@ -136,6 +157,16 @@ class MixerSpec:
     norm_alpha: list = field(default_factory=lambda: [0.0, 0.0, 0.0, 0.0])   # norm1, norm1b, norm2, norm2b (read from the checkpoint)
     side_dim: int = 0
     side_col: int = 0
+    # sink_attention: pooled blocks in front of the window, chunks of fixed places, a soft cap, a sink of score zero, norms with gains in
+    # front of the rotation, unit-RMS values; blocks without norms in front of their sublayers; a side mixer added with constant factors
+    pool: int = 0
+    chunk: int = 0
+    softcap: float = 0.0
+    sink_zero: bool = False
+    qk_norm: bool = False
+    v_unit: bool = False
+    branch_scale: float = 0.0
+    pre_norms: bool = True
 
     @property
     def inner(self) -> int:
@@ -185,6 +216,7 @@ class Config:
     loop_mode: str = "step"           # in front of every pass: "step" (x += [x0] + vector), "none", "project" (x <- W [x; x0])
     token_side_dim: int = 0           # > 0: a per-layer token input of that width (table `side.embed` [vocab, layers * dim])
     final_norm_kind: int = 0          # 1: the final norm is the squashing norm
+    embed_norm: bool = False          # the stream starts with an RMS norm of the token embedding (gain `embed.norm`)
 
     def layer_variant(self, i: int, max_seq: Optional[int] = None) -> dict:
         """Norm placement and attention mode of layer ``i``, as the reference's per-architecture block.rs sets them up:
@@ -216,7 +248,7 @@ class Config:
     @property
     def layer_list(self) -> bool:
         """The checkpoint's config lists its layers one by one; such models keep an fp32 residual stream."""
-        return self.block_kind in ("nigenex", "setodra", "nuvarax", "netolorn")
+        return self.block_kind in ("nigenex", "setodra", "nuvarax", "netolorn", "mafosun")
 
     @property
     def scalar_final_norm(self) -> bool:
@@ -447,6 +479,84 @@ class Config:
                       head_dim=specs[0].vdim, max_seq_len=int(max_seq), block_kind="netolorn", layers=specs, model_prefix="", loop=loop,
                       loop_mode="project", token_side_dim=side, final_norm_kind=1)
 
+    @staticmethod
+    def _from_mafosun(d: dict, max_seq: int = 4096) -> "Config":
+        """Mafosun ``config.json``: ``width``, ``vocab``, ``norm.eps`` and ``layers``, whose entries give ``type`` (``attention``: grouped-query
+        attention with ``rot`` (dims, base, scaling), ``mask`` (size, pool), ``scale``, ``softcap``; ``parallel``: chunked attention
+        (``mixer.left``: ``mask.size``, ``scale``) beside retention (``mixer.right``: ``decay``, ``rot``), added with ``left_scale`` and
+        ``right_scale``), the mixer's sizes and the feed-forward (``mlp``: kind ``dense`` with ``ff``; kind ``moe`` with ``router`` (experts, top,
+        groups.{count, keep}) and ``expert.ff``; or null).  Sublayers read the stream itself; their outputs are RMS-normed; the output
+        projection is the embedding table."""
+        specs = []
+        for i, L in enumerate(d["layers"]):
+            kind, m = L.get("type"), L["mixer"]
+
+            def attention(m, **kw):
+                return MixerSpec(type="sink_attention", heads=int(m["heads"]), kv_heads=int(m.get("kv_heads") or m["heads"]), dim=int(m["dim"]),
+                                 vdim=int(m.get("vdim") or m["dim"]), scale=float(m["scale"]), softcap=float(m.get("softcap") or 0.0), qk_norm=True, **kw)
+
+            if kind == "attention":
+                mask = m.get("mask") or {}
+                size = int(mask.get("size") or 0)
+                sp = attention(m, rot=RotarySpec.stretched(m.get("rot"), True), window=size, pool=int(mask.get("pool") or 0) if size else 0, sink_zero=True)
+            elif kind == "parallel":
+                a, b = m["left"], m["right"]
+                side = MixerSpec(type="retention", heads=int(b["heads"]), dim=int(b["dim"]), vdim=int(b.get("vdim") or b["dim"]),
+                                 decay=[float(x) for x in b["decay"]], rot=RotarySpec.stretched(b.get("rot"), False), branch_scale=float(m["right_scale"]))
+                if len(side.decay) != side.heads:
+                    raise ValueError(f"layer {i}: {len(side.decay)} decays for {side.heads} heads")
+                if side.rot.dims > side.dim:
+                    raise ValueError(f"layer {i}: rot.dims {side.rot.dims} above dim {side.dim}")
+                sp = attention(a, chunk=int((a.get("mask") or {}).get("size") or 0), v_unit=True, branch_scale=float(m["left_scale"]), side=side)
+            else:
+                raise ValueError(f"layer {i}: mixer type {kind!r} is not part of this design")
+            if sp.heads % sp.n_kv:
+                raise ValueError(f"layer {i}: {sp.heads} heads over {sp.n_kv} key heads")
+            if sp.rot.dims > sp.dim:
+                raise ValueError(f"layer {i}: rot.dims {sp.rot.dims} above dim {sp.dim}")
+            mlp = L.get("mlp")
+            if mlp is not None:
+                if mlp.get("kind") == "dense":
+                    sp.dense_ff, sp.dense_act = int(mlp["ff"]), 3
+                elif mlp.get("kind") == "moe":
+                    r, g = mlp["router"], mlp["router"].get("groups") or {}
+                    sp.moe = MoeSpec(experts=int(r["experts"]), top=int(r["top"]), ff=int(mlp["expert"]["ff"]), groups=int(g.get("count") or 1),
+                                     groups_keep=int(g.get("keep") or 1), plain_weights=True)
+                    if sp.moe.experts % sp.moe.groups or sp.moe.top > sp.moe.groups_keep * (sp.moe.experts // sp.moe.groups):
+                        raise ValueError(f"layer {i}: top {sp.moe.top} of {sp.moe.experts} experts in {sp.moe.groups} groups, {sp.moe.groups_keep} kept")
+                else:
+                    raise ValueError(f"layer {i}: feed-forward kind {mlp.get('kind')!r} is not part of this design")
+            sp.pre_norms, sp.post_norms = False, True
+            specs.append(sp)
+        if not specs:
+            raise ValueError("config lists no layers")
+        return Config(hidden_size=int(d["width"]), intermediate_size=0, vocab_size=int(d["vocab"]), num_hidden_layers=len(specs),
+                      num_attention_heads=specs[0].heads, num_key_value_heads=specs[0].n_kv, rms_norm_eps=float(d["norm"]["eps"]),
+                      head_dim=specs[0].vdim, max_seq_len=int(max_seq), block_kind="mafosun", layers=specs, model_prefix="",
+                      loop_injects=False, tie_word_embeddings=True, embed_norm=True)
+
+    def to_mafosun(self) -> dict:
+        """The ``config.json`` of a Mafosun Config (inverse of ``_from_mafosun``)."""
+        layers = []
+        for s in self.layers:
+            att = {"heads": s.heads, "kv_heads": s.n_kv, "dim": s.dim, "vdim": s.vdim, "scale": s.scale}
+            if s.side is None:
+                kind, m = "attention", dict(att, rot=s.rot.to_dict(), softcap=s.softcap or None,
+                                            mask={"size": s.window, "pool": s.pool} if s.window else None)
+            else:
+                r = s.side
+                kind, m = "parallel", {"left": dict(att, mask={"size": s.chunk} if s.chunk else None), "left_scale": s.branch_scale,
+                                       "right": {"heads": r.heads, "dim": r.dim, "vdim": r.vdim, "decay": list(r.decay), "rot": r.rot.to_dict()},
+                                       "right_scale": r.branch_scale}
+            mo = s.moe
+            if mo is not None:
+                mlp = {"kind": "moe", "router": {"experts": mo.experts, "top": mo.top, "groups": {"count": mo.groups, "keep": mo.groups_keep}},
+                       "expert": {"ff": mo.ff}}
+            else:
+                mlp = {"kind": "dense", "ff": s.dense_ff} if s.dense_ff else None
+            layers.append({"type": kind, "mixer": m, "mlp": mlp})
+        return {"architecture": "Mafosun", "width": self.hidden_size, "vocab": self.vocab_size, "norm": {"eps": self.rms_norm_eps}, "layers": layers}
+
     def to_netolorn(self) -> dict:
         """The ``config.json`` of a Netolorn Config (inverse of ``_from_netolorn``)."""
         layers = []
@@ -529,6 +639,8 @@ class Config:
             return Config._from_nuvarax(d)
         if d.get("architecture") == "Netolorn":
             return Config._from_netolorn(d)
+        if d.get("architecture") == "Mafosun":
+            return Config._from_mafosun(d)
         arch = Config.detect_arch(d)
         if arch in Config._OTHER_BLOCKS:
             raise ValueError(f"architecture {arch!r} is outside the block-forward path built here")
@@ -619,6 +731,8 @@ class Config:
             return self.to_nuvarax()
         if self.block_kind == "netolorn":
             return self.to_netolorn()
+        if self.block_kind == "mafosun":
+            return self.to_mafosun()
         d = dict(
             architectures=[arch], hidden_size=self.hidden_size, intermediate_size=self.intermediate_size,
             vocab_size=self.vocab_size, num_hidden_layers=self.num_hidden_layers,

@@ -39,6 +39,11 @@ struct WinAttn {
   const void *sink;      // [heads] D: a logit that joins every row's denominator, without key or value
   const void *gate;      // gate_mode 1: [B*S, ldg] D logits, one per head at column h; 2: one per output element at h*hd + i
   int gate_mode, ldg;
+  // pooled blocks (rows of the second pair of tensor maps): block blk of `pool` positions is one more key once (blk + 1) pool <=
+  // i - window + 1; chunk: keys of the row's own chunk of that many positions only; sink_zero: the denominator holds exp(0);
+  // out_scale: a constant factor of the output
+  int pool, chunk, sink_zero;
+  float out_scale = 1.f;
 };
 constexpr int WA_MAX_HD = 256;
 

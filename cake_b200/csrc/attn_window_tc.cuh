@@ -5,7 +5,8 @@
 //     exponent constant is log2 e), rows that see nothing in a tile keeping a -inf reference,
 //   * the K tensor map given twice: the keys double as values, the V ring is filled from the same cache rows,
 //   * the head gate and the caller's row stride in the epilogue,
-//   * optionally: the tiles of the kept first keys ahead of the window's tiles, a sink logit in the denominator, a gate per head
+//   * optionally: the tiles of pooled blocks (tensor maps of their own) and of the kept first keys ahead of the window's tiles, chunks
+//     of fixed places instead of or beside the window, a sink logit in the denominator, a gate per head
 //     or per output element from a buffer of its own, and key / value buffers whose first row is a later position (key0).
 // Warp roles, barriers, TMEM layout and the P_hi + P_lo operand are those of attn_prefill_tc_kernel; see there.
 // Cost model: four MUFU operations per score (tanh = ex2 + rcp, ln, the softmax's ex2) against one in the plain kernel make
@@ -19,7 +20,8 @@ namespace cake {
 template <typename T>
 __global__ void __launch_bounds__(FT_THREADS, 2)
 attn_window_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant__ CUtensorMap map_k,
-                      const __grid_constant__ CUtensorMap map_v, const WinAttn p, float tau_log2) {
+                      const __grid_constant__ CUtensorMap map_v, const __grid_constant__ CUtensorMap map_pk,
+                      const __grid_constant__ CUtensorMap map_pv, const WinAttn p, float tau_log2) {
   const int S = p.S, n_heads = p.heads, n_kv = p.n_kv, pos0 = p.pos0;
   constexpr float scale_log2 = 1.4426950408889634f;  // the modified score is in natural units: p = 2^((s - m) log2 e)
   extern __shared__ unsigned char ft_smem_raw[];
@@ -38,10 +40,13 @@ attn_window_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_co
   const int m0 = mt * FT_BM;
   const int kv_end = pos0 + min(S, m0 + FT_BM);  // keys visible to the last query of this tile
   // tiles [j_lo, j_end): from the one that holds the first key the tile's first row sees; rings and phases count from j_lo
-  const int j_lo = p.window > 0 ? max(0, pos0 + m0 - p.window + 1) / FT_BN : 0;
-  // kept first keys that lie before the window's first tile come first: iteration j works on key tile j (j < n_kept) or
-  // j_lo + j - n_kept
-  const int n_kept = min(j_lo, (p.keep_first + FT_BN - 1) / FT_BN);
+  int k_lo = p.window > 0 ? max(0, pos0 + m0 - p.window + 1) : 0;
+  if (p.chunk > 0) k_lo = max(k_lo, (pos0 + m0) / p.chunk * p.chunk);
+  const int j_lo = k_lo / FT_BN;
+  // pooled blocks seen by the tile's last row come first (iterations j < n_pool), then kept first keys that lie before the
+  // window's first tile (key tile j - n_pool for j < n_kept), then the window's tiles (j_lo + j - n_kept)
+  const int n_pool = p.pool > 0 && kv_end > p.window ? ((kv_end - p.window) / p.pool + FT_BN - 1) / FT_BN : 0;
+  const int n_kept = n_pool + min(j_lo, (p.keep_first + FT_BN - 1) / FT_BN);
   const int n_tiles = n_kept + (kv_end + FT_BN - 1) / FT_BN - j_lo;
   const int j_add = j_lo - n_kept;
 
@@ -77,13 +82,15 @@ attn_window_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_co
         unsigned char *kd = k_s + st * FT_KV_BYTES, *vd = v_s + st * FT_KV_BYTES;
         if (j >= 2) mbar_wait(&k_empty[st], eph);
         mbar_arrive_expect_tx(&k_full[st], FT_KV_BYTES);
-        const int krow = (j < n_kept ? j : j + j_add) * FT_BN - p.key0;  // rows before the buffer read as zeros and are masked
-        tma_load_3d(kd, &map_k, 0, krow, slab, &k_full[st]);
-        tma_load_3d(kd + FT_KV_BYTES / 2, &map_k, 64, krow, slab, &k_full[st]);
+        const bool pooled = j < n_pool;
+        const CUtensorMap *mk = pooled ? &map_pk : &map_k, *mv = pooled ? &map_pv : &map_v;
+        const int krow = pooled ? j * FT_BN : (j < n_kept ? j - n_pool : j + j_add) * FT_BN - p.key0;  // rows before the buffer read as zeros and are masked
+        tma_load_3d(kd, mk, 0, krow, slab, &k_full[st]);
+        tma_load_3d(kd + FT_KV_BYTES / 2, mk, 64, krow, slab, &k_full[st]);
         if (j >= 2) mbar_wait(&v_empty[st], eph);
         mbar_arrive_expect_tx(&v_full[st], FT_KV_BYTES);
-        tma_load_3d(vd, &map_v, 0, krow, slab, &v_full[st]);
-        tma_load_3d(vd + FT_KV_BYTES / 2, &map_v, 64, krow, slab, &v_full[st]);
+        tma_load_3d(vd, mv, 0, krow, slab, &v_full[st]);
+        tma_load_3d(vd + FT_KV_BYTES / 2, mv, 64, krow, slab, &v_full[st]);
       }
     }
   } else if (warp == 5) {
@@ -137,6 +144,10 @@ attn_window_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_co
     const float r1 = biased ? DT<T>::to_f(reinterpret_cast<const T *>(p.r1)[h]) : 0.f;
     const float r2 = biased ? DT<T>::to_f(reinterpret_cast<const T *>(p.r2)[h]) : 0.f;
     const float inv_cap2 = p.softcap > 0.f ? 2.0f / p.softcap : 0.f;
+    // this row's reach: its window and its chunk; the pooled blocks it sees (blocks [0, seen))
+    const float row_win = p.chunk > 0 ? fminf(p.window > 0 ? (float)p.window : 3.0e38f, (float)(qp % p.chunk + 1))
+                                      : p.window > 0 ? (float)p.window : 3.0e38f;
+    const int seen = p.pool > 0 && qp >= p.window ? (qp - p.window + 1) / p.pool : 0;
     for (int j = 0; j < n_tiles; j++) {
       const uint32_t tmem_sp = tmem_base + lane_addr + (uint32_t)((j & 1) * 64);
       mbar_wait(&s_full[j & 1], (uint32_t)(j >> 1) & 1u);
@@ -156,8 +167,10 @@ attn_window_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_co
       // the distance is carried as a float (exact below 2^24, no I2F on the MUFU pipe), masked entries take the arithmetic
       // with a clamped distance and are replaced by -inf at the end.
       float mx = -INFINITY;
-      const float fd0 = (float)(qp - (j < n_kept ? j : j + j_add) * FT_BN);  // distance to the tile's first key
-      const float fwin = p.window > 0 ? (float)p.window : 3.0e38f;
+      // distance to the tile's first key; in a tile of pooled blocks "distance" counts back from the last block that the row sees
+      const bool pooled = j < n_pool;
+      const float fd0 = pooled ? (float)(seen - 1 - j * FT_BN) : (float)(qp - (j < n_kept ? j - n_pool : j + j_add) * FT_BN);
+      const float fwin = pooled ? 3.0e38f : row_win;
       const float fkept = (float)(qp - p.keep_first);  // key < keep_first  <=>  distance > qp - keep_first
 #pragma unroll
       for (int i = 0; i < FT_BN; i++) {
@@ -231,7 +244,8 @@ attn_window_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_co
       gate = 1.0f / (1.0f + expf(-DT<T>::to_f(reinterpret_cast<const T *>(p.qkg)[(size_t)(b * S + t) * p.ld + p.gate_col + h])));
     // the sink counts once in the denominator, relative to the row's reference maximum (which holds at least the row's own key)
     if (p.sink) l_run += expf(DT<T>::to_f(reinterpret_cast<const T *>(p.sink)[h]) - m_run);
-    const float inv = gate / l_run;
+    if (p.sink_zero) l_run += expf(-m_run);
+    const float inv = gate * p.out_scale / l_run;
     T *dst = reinterpret_cast<T *>(p.y) + (size_t)(b * S + t) * p.ldy + h * FT_HD;
 #pragma unroll 1
     for (int c0 = 0; c0 < FT_HD; c0 += 32) {

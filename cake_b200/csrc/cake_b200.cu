@@ -160,6 +160,7 @@ struct cake_b200_ctx {
   void *side_tab = nullptr, *ln_f_b = nullptr;
   int side_cols = 0, final_norm_kind = 0;
   float final_alpha = 0.f;
+  void *embed_norm = nullptr;  // gain of the norm behind the token embedding
   size_t d_ids_n = 0;
   // cake_b200_stream_project: the projection [hidden, 2 hidden] and its operand [rows, 2 hidden] in D
   void *proj_w = nullptr, *proj_ws = nullptr;
@@ -242,6 +243,10 @@ struct cake_b200_block {
   void *m_sink = nullptr, *m_dq_norm = nullptr, *m_uq = nullptr;
   void *ln1_b = nullptr, *post1_b = nullptr, *ln2_b = nullptr, *post2_b = nullptr;
   void *sd_gate = nullptr, *sd_proj = nullptr, *sd_norm = nullptr;
+  void *m_qn = nullptr, *m_kn = nullptr;  // sink attention with qk_norm: gains [dim]
+  // a side mixer that is added with constant factors: wo is [hidden, inner | side inner], one output projection for both
+  bool joint = false;
+  float out_scale = 1.f;
   bool variant() const { return !ln1 || !ln2 || pan || pfn || window >= 0 || !use_rope || ctx->cfg.pre_reshape_qk_norm; }
 };
 
@@ -265,6 +270,7 @@ struct cake_b200_cache {
   // side mixer; rec_aux: the normaliser and running maximum of a matrix memory [batch, heads, dk + 1] fp32; canon_hist: the
   // last canon_taps - 1 normed inputs of the block [batch, taps - 1, hidden] fp32
   std::vector<float *> rec_aux, canon_hist;
+  std::vector<void *> pk, pv;  // sink attention with pooled blocks: their keys and values, [batch, kv_heads, cap / pool, dim | vdim]
   std::vector<void *> vt;   // talking attention on the tensor cores: the values once more, [batch, kv_heads, vdim, cap_t] with positions innermost
   // cake_b200_embed_at: the last token of every batch row and the position the embedding has reached
   std::vector<uint32_t> last_tok;
@@ -592,7 +598,7 @@ extern "C" void cake_b200_ctx_destroy(cake_b200_ctx *c) {
     if (b) cudaFree(b);
   if (c->bigram) cudaFree(c->bigram);
   if (c->pos_tab) cudaFree(c->pos_tab);
-  for (void *b : {c->side_tab, c->ln_f_b, c->proj_w, c->proj_ws})
+  for (void *b : {c->side_tab, c->ln_f_b, c->proj_w, c->proj_ws, c->embed_norm})
     if (b) cudaFree(b);
   for (void *b : c->inject_vec)
     if (b) cudaFree(b);
@@ -784,7 +790,7 @@ extern "C" void cake_b200_block_free(cake_b200_block *b) {
                   b->w_in, b->w_out, b->g, b->shift, b->r1, b->r2, b->m_dkv_norm, b->m_uk, b->m_uv, b->m_ukt, b->m_conv, b->m_conv_b, b->m_dt_bias,
                   b->m_a_log, b->m_d, b->m_norm, b->m_router, b->m_corr, b->m_eg, b->m_ed, b->m_cos, b->m_sin, b->m_decay,
                   b->post1, b->post2, b->canon, b->b_in, b->m_ob, b->m_talk, b->m_branch, b->m_ib, b->m_fb, b->m_bias,
-                  b->m_sink, b->m_dq_norm, b->m_uq, b->ln1_b, b->post1_b, b->ln2_b, b->post2_b, b->sd_gate, b->sd_proj, b->sd_norm};
+                  b->m_sink, b->m_dq_norm, b->m_uq, b->ln1_b, b->post1_b, b->ln2_b, b->post2_b, b->sd_gate, b->sd_proj, b->sd_norm, b->m_qn, b->m_kn};
   for (void *p : bufs)
     if (p) cudaFree(p);  // cudaFree synchronises with outstanding work
   if (b->side) cake_b200_block_free(b->side);
@@ -826,6 +832,8 @@ extern "C" int cake_b200_cache_create(cake_b200_ctx *c, int batch, int max_seq, 
   k->kv_hd.assign(slots, 0);
   k->rec_aux.assign(slots, nullptr);
   k->vt.assign(slots, nullptr);
+  k->pk.assign(slots, nullptr);
+  k->pv.assign(slots, nullptr);
   k->canon_hist.assign(c->cfg.n_layers, nullptr);
   k->last_tok.assign(batch, 0);
   k->shift_state[0].assign(c->cfg.n_layers, nullptr);
@@ -889,6 +897,10 @@ extern "C" void cake_b200_cache_free(cake_b200_cache *k) {
   for (float *p : k->rec_aux)
     if (p) cudaFree(p);
   for (void *p : k->vt)
+    if (p) cudaFree(p);
+  for (void *p : k->pk)
+    if (p) cudaFree(p);
+  for (void *p : k->pv)
     if (p) cudaFree(p);
   for (float *p : k->canon_hist)
     if (p) cudaFree(p);
@@ -1538,13 +1550,15 @@ template <typename T> static int listed_attention_tc(cake_b200_ctx *c, const Win
   RC(make_tmap3(&mk, wa.kc, (uint64_t)wa.hd, (uint64_t)wa.hd, (uint64_t)(wa.pos0 + wa.S), (uint64_t)wa.cap, (uint64_t)wa.B * wa.n_kv, c->cfg.dtype, FT_BN));
   dim3 gt((wa.S + FT_BM - 1) / FT_BM, wa.heads, wa.B);
   *done = true;
-  return launch_pdl(c, attn_window_tc_kernel<T>, gt, dim3(FT_THREADS), (size_t)FT_SMEM_BYTES, mq, mk, mk, wa, fa_tau * 1.4426950408889634f);
+  return launch_pdl(c, attn_window_tc_kernel<T>, gt, dim3(FT_THREADS), (size_t)FT_SMEM_BYTES, mq, mk, mk, mk, mk, wa, fa_tau * 1.4426950408889634f);
 }
 template <> int listed_attention_tc<float>(cake_b200_ctx *, const WinAttn &, bool *done) { *done = false; return CAKE_B200_OK; }
 // attn_window_tc_kernel with its optional parts (kept first keys, sink, a gate buffer, buffers that start at key0).
 // kv_row: 0 = kc / vc are caches [B, n_kv, cap, 128]; > 0 = they hold rows of that many elements with the heads side by side
 // (one batch row; rows = positions key0 ..).
-template <typename T> static int window_attention_tc(cake_b200_ctx *c, const WinAttn &wa, int kv_row, uint64_t *lc) {
+// pk / pv: the caches of pooled blocks [B, n_kv, pcap, 128] (wa.pool > 0).
+template <typename T> static int window_attention_tc(cake_b200_ctx *c, const WinAttn &wa, int kv_row, uint64_t *lc, const void *pk = nullptr,
+                                                     const void *pv = nullptr, int pcap = 0) {
   static const float fa_tau = []() { const char *e = getenv("CAKE_B200_FA_TAU"); return e ? (float)atof(e) : 5.545f; }();
   if (wa.hd != FT_HD || wa.ldy % 8 != 0 || wa.ld % 8 != 0 || (kv_row && wa.B != 1) || (wa.gate_mode == 2 && (wa.ldg % 8 != 0 || ((uintptr_t)wa.gate & 15) != 0)))
     return fail(CAKE_B200_EINVAL, "window attention on the tensor cores: shapes not supported");
@@ -1558,11 +1572,17 @@ template <typename T> static int window_attention_tc(cake_b200_ctx *c, const Win
     RC(make_tmap3(&mk, wa.kc, (uint64_t)FT_HD, (uint64_t)FT_HD, vis, (uint64_t)wa.cap, (uint64_t)wa.B * wa.n_kv, c->cfg.dtype, FT_BN));
     RC(make_tmap3(&mv, wa.vc, (uint64_t)FT_HD, (uint64_t)FT_HD, vis, (uint64_t)wa.cap, (uint64_t)wa.B * wa.n_kv, c->cfg.dtype, FT_BN));
   }
+  CUtensorMap mpk = mk, mpv = mv;
+  const int n_blocks = wa.pool > 0 ? (wa.pos0 + wa.S) / wa.pool : 0;  // complete ones; every block that a row sees is
+  if (n_blocks > 0) {
+    RC(make_tmap3(&mpk, pk, (uint64_t)FT_HD, (uint64_t)FT_HD, (uint64_t)n_blocks, (uint64_t)pcap, (uint64_t)wa.B * wa.n_kv, c->cfg.dtype, FT_BN));
+    RC(make_tmap3(&mpv, pv, (uint64_t)FT_HD, (uint64_t)FT_HD, (uint64_t)n_blocks, (uint64_t)pcap, (uint64_t)wa.B * wa.n_kv, c->cfg.dtype, FT_BN));
+  }
   dim3 gt((wa.S + FT_BM - 1) / FT_BM, wa.heads, wa.B);
   (void)lc;  // launch_pdl counts
-  return launch_pdl(c, attn_window_tc_kernel<T>, gt, dim3(FT_THREADS), (size_t)FT_SMEM_BYTES, mq, mk, mv, wa, fa_tau * 1.4426950408889634f);
+  return launch_pdl(c, attn_window_tc_kernel<T>, gt, dim3(FT_THREADS), (size_t)FT_SMEM_BYTES, mq, mk, mv, mpk, mpv, wa, fa_tau * 1.4426950408889634f);
 }
-template <> int window_attention_tc<float>(cake_b200_ctx *, const WinAttn &, int, uint64_t *) { return CAKE_B200_EINVAL; }
+template <> int window_attention_tc<float>(cake_b200_ctx *, const WinAttn &, int, uint64_t *, const void *, const void *, int) { return CAKE_B200_EINVAL; }
 // steps of a few tokens in 16-bit D with 16-byte rows: eight lanes per key (attn_window_decode_vec_kernel)
 template <typename T> static int listed_attention_vec(cake_b200_ctx *c, const WinAttn &wa, bool *done) {
   *done = false;
@@ -1693,6 +1713,17 @@ static void mixer_rope_tables(const cake_b200_rotary_spec &r, int rows, std::vec
     }
     amp = 0.1 * log(r.yarn_factor) + 1.0;
   }
+  if (r.stretch_factor > 0.0) {
+    for (int i = 0; i < half; i++) {
+      const double l = 2.0 * 3.14159265358979323846 / f[i];
+      if (l < r.stretch_original / r.stretch_high) continue;
+      if (l > r.stretch_original / r.stretch_low) f[i] /= r.stretch_factor;
+      else {
+        const double s = (r.stretch_original / l - r.stretch_low) / (r.stretch_high - r.stretch_low);
+        f[i] = (1.0 - s) * f[i] / r.stretch_factor + s * f[i];
+      }
+    }
+  }
   cs.resize((size_t)rows * half);
   sn.resize((size_t)rows * half);
   for (int p = 0; p < rows; p++)
@@ -1707,7 +1738,7 @@ static void mixer_rope_tables(const cake_b200_rotary_spec &r, int rows, std::vec
 static int load_routed_ff(cake_b200_ctx *c, cake_b200_block *b, const cake_b200_moe_spec &mo, const cake_b200_mixer_tensors *t, int layer_idx) {
   const size_t es = c->es, H = c->cfg.hidden;
   const size_t E = mo.experts, Et = E + mo.identity, I = mo.ff, Is = mo.shared_ff;
-  RC(upload(c, &b->ln2, t->norm2, H * es));
+  if (t->norm2) RC(upload(c, &b->ln2, t->norm2, H * es));
   // router rows, then the shared expert's gate vector as one more row, zero rows up to the tensor-core tile: one product
   // gives every logit of a token
   const size_t NP = (size_t)round_up((int)Et + 1, TC_BN);
@@ -1716,7 +1747,7 @@ static int load_routed_ff(cake_b200_ctx *c, cake_b200_block *b, const cake_b200_
   CU(cudaStreamSynchronize(0));
   RC(pipe_copy(c, b->m_router, Et * H * es, t->router, Et * H * es, Et * H * es, 1));
   if (Is) RC(pipe_copy(c, (char *)b->m_router + Et * H * es, H * es, t->s_sg, H * es, H * es, 1));
-  RC(upload(c, &b->m_corr, t->correction, Et * es));
+  if (t->correction) RC(upload(c, &b->m_corr, t->correction, Et * es));
   if (E) {
     // all experts stacked: gate / up row-interleaved per expert (as the dense blocks lay theirs out) and the down matrices,
     // so that a grouped product addresses expert e at row e * N of one matrix
@@ -1746,7 +1777,7 @@ extern "C" int cake_b200_block_load_mixer(cake_b200_ctx *c, int layer_idx, const
   if (!c || !sp || !t || !out) return fail(CAKE_B200_EINVAL, "null argument");
   if (!c->cfg.layer_list) return fail(CAKE_B200_EINVAL, "block_load_mixer needs a ctx created with layer_list = 1");
   if (mixer_kind_ext(sp->kind) || sp->side || sp->norm_offset != 0.f || sp->canon_taps > 0 || sp->dense_ff > 0 || t->post1 || t->post2 ||
-      sp->norm_kind != 0 || sp->side_dim > 0)
+      sp->norm_kind != 0 || sp->side_dim > 0 || sp->moe.groups > 1 || sp->moe.plain_weights || sp->rot.interleaved)
     return load_mixer_ext(c, layer_idx, sp, t, out);
   const cake_b200_moe_spec &mo = sp->moe;
   const bool has_ff = mo.experts + mo.identity > 0;
@@ -1858,13 +1889,28 @@ static int distance_bucket(int n, int rows, double dmax) {
 
 struct InPart { const void *w; size_t rows; const void *bias; };
 // validates one mixer of an ext block, uploads its own tensors into `b` and appends its projections to the fused input product
+// (joint: the output projection is one matrix of the whole block, uploaded by the caller)
 static int load_sub_mixer(cake_b200_ctx *c, cake_b200_block *b, const cake_b200_mixer_spec *sp, const cake_b200_mixer_tensors *t,
-                          std::vector<InPart> &parts, size_t &row, int layer_idx) {
+                          std::vector<InPart> &parts, size_t &row, int layer_idx, bool joint) {
   const size_t es = c->es, H = c->cfg.hidden;
   if (sp->heads < 1 || sp->vdim < 1 || sp->dim < 1 || !t->o) return fail(CAKE_B200_EINVAL, "layer %d: bad heads / dim / vdim or null o", layer_idx);
   const int G = sub_kv_heads(*sp);
   if (G < 1 || sp->heads % G) return fail(CAKE_B200_EINVAL, "layer %d: %d heads over %d key heads", layer_idx, sp->heads, G);
   const size_t inner = (size_t)sp->heads * sp->vdim;
+  const cake_b200_rotary_spec &ro = sp->rot;
+  if (ro.dims < 0 || ro.dims % 2 || (ro.dims > 0 && !(ro.base > 0.0)) ||
+      (ro.stretch_factor > 0.0 && (!(ro.stretch_low > 0.0) || !(ro.stretch_high > ro.stretch_low) || !(ro.stretch_original > 0.0) || ro.yarn_factor > 0.0)))
+    return fail(CAKE_B200_EINVAL, "layer %d: bad rotation", layer_idx);
+  auto rope_tables = [&]() -> int {
+    if (ro.dims < 2) return CAKE_B200_OK;
+    std::vector<float> cs, sn;
+    b->m_rope_rows = c->cfg.max_seq;
+    mixer_rope_tables(ro, b->m_rope_rows, cs, sn);
+    RC(upload(c, (void **)&b->m_cos, cs.data(), cs.size() * sizeof(float)));
+    RC(upload(c, (void **)&b->m_sin, sn.data(), sn.size() * sizeof(float)));
+    CU(cudaStreamSynchronize(c->load_stream));  // the staging copy has left the vectors
+    return CAKE_B200_OK;
+  };
   auto align8 = [&]() {
     const size_t pad = (8 - row % 8) % 8;
     if (pad) { parts.push_back({nullptr, pad, nullptr}); row += pad; }
@@ -1879,7 +1925,7 @@ static int load_sub_mixer(cake_b200_ctx *c, cake_b200_block *b, const cake_b200_
   b->ms.decay = nullptr;
   b->ms.side = nullptr;
   b->ms.kv_heads = G;
-  RC(upload(c, &b->wo, t->o, H * inner * es));
+  if (!joint) RC(upload(c, &b->wo, t->o, H * inner * es));
   if (t->branch_norm) RC(upload(c, &b->m_branch, t->branch_norm, H * es));
   if (sp->kind == CAKE_B200_MIX_DELTA) {
     if (sp->conv < 1 || !t->q || !t->k || !t->v || !t->g || !t->q_conv || !t->k_conv || !t->v_conv || !t->beta || !t->a_proj || !t->a_log || !t->dt_bias || !t->norm)
@@ -1961,10 +2007,18 @@ static int load_sub_mixer(cake_b200_ctx *c, cake_b200_block *b, const cake_b200_
     RC(upload(c, &b->m_fb, t->f_b, sp->heads * es));
     RC(upload(c, &b->m_norm, t->norm, inner * es));
   } else if (sp->kind == CAKE_B200_MIX_SINK_ATTENTION) {
-    if (!t->q || !t->k || !t->v || sp->window < 0 || sp->keep_first < 0 || sp->rot.dims < 0 || sp->rot.dims % 2 || sp->rot.dims > sp->dim ||
-        (sp->rot.dims > 0 && !(sp->rot.base > 0.0)))
+    if (!t->q || !t->k || !t->v || sp->window < 0 || sp->keep_first < 0 || sp->rot.dims > sp->dim)
       return fail(CAKE_B200_EINVAL, "layer %d: sink attention needs q / k / v, window and keep_first >= 0 and an even rot.dims <= dim", layer_idx);
     if (std::max(sp->dim, sp->vdim) > 768) return fail(CAKE_B200_EINVAL, "layer %d: head sizes above 768", layer_idx);
+    if (sp->pool < 0 || sp->chunk < 0 || sp->softcap < 0.f || (sp->pool > 0 && (sp->window < 1 || sp->chunk > 0 || sp->keep_first > 0)))
+      return fail(CAKE_B200_EINVAL, "layer %d: pooled blocks need a window and stand beside neither chunks nor kept first tokens", layer_idx);
+    if (sp->qk_norm && (sp->qk_unit || !t->q_norm || !t->k_norm))
+      return fail(CAKE_B200_EINVAL, "layer %d: qk_norm needs q_norm / k_norm and excludes qk_unit", layer_idx);
+    if (sp->sink_zero && t->sink) return fail(CAKE_B200_EINVAL, "layer %d: a learned sink and the zero sink exclude each other", layer_idx);
+    if (sp->qk_norm) {
+      RC(upload(c, &b->m_qn, t->q_norm, (size_t)sp->dim * es));
+      RC(upload(c, &b->m_kn, t->k_norm, (size_t)sp->dim * es));
+    }
     align8();
     b->pc[0] = add(t->q, (size_t)sp->heads * sp->dim, t->q_b);
     align8();
@@ -1976,14 +2030,21 @@ static int load_sub_mixer(cake_b200_ctx *c, cake_b200_block *b, const cake_b200_
       b->pc[3] = add(t->g, inner, nullptr);
     } else b->pc[3] = -1;
     if (t->sink) RC(upload(c, &b->m_sink, t->sink, (size_t)sp->heads * es));
-    if (sp->rot.dims > 0) {
-      std::vector<float> cs, sn;
-      b->m_rope_rows = c->cfg.max_seq;
-      mixer_rope_tables(sp->rot, b->m_rope_rows, cs, sn);
-      RC(upload(c, (void **)&b->m_cos, cs.data(), cs.size() * sizeof(float)));
-      RC(upload(c, (void **)&b->m_sin, sn.data(), sn.size() * sizeof(float)));
-      CU(cudaStreamSynchronize(c->load_stream));  // the staging copy has left the vectors
-    }
+    RC(rope_tables());
+  } else if (sp->kind == CAKE_B200_MIX_RETENTION) {
+    if (!t->q || !t->k || !t->v || !t->g || !sp->decay || ro.dims > sp->dim || ro.interleaved || G != sp->heads)
+      return fail(CAKE_B200_EINVAL, "layer %d: retention needs q / k / v / g, decay, rot.dims <= dim (pairs half the rotated width apart) and a key head per head", layer_idx);
+    const size_t qk = (size_t)sp->heads * sp->dim;
+    align8();
+    b->pc[0] = add(t->q, qk, nullptr);
+    align8();
+    b->pc[1] = add(t->k, qk, nullptr);
+    align8();
+    b->pc[2] = add(t->v, inner, nullptr);
+    align8();
+    b->pc[3] = add(t->g, inner, nullptr);
+    RC(upload(c, (void **)&b->m_decay, sp->decay, sp->heads * sizeof(float)));
+    RC(rope_tables());
   } else if (sp->kind == CAKE_B200_MIX_LATENT_WINDOW) {
     if (sp->q_rank < 1 || sp->kv_rank < 1 || sp->kv_rank > 768 || sp->window < 0 || sp->keep_first < 0 || !t->dq || !t->dq_norm || !t->uq || !t->dkv ||
         !t->dkv_norm || !t->uk || !t->uv)
@@ -2007,14 +2068,19 @@ static int load_sub_mixer(cake_b200_ctx *c, cake_b200_block *b, const cake_b200_
 }
 
 static int load_mixer_ext(cake_b200_ctx *c, int layer_idx, const cake_b200_mixer_spec *sp, const cake_b200_mixer_tensors *t, cake_b200_block **out) {
-  if (!t->norm1) return fail(CAKE_B200_EINVAL, "layer %d: null norm1", layer_idx);
+  // without norm1 / norm2 the sublayers read the stream itself and only their outputs are normed
+  const bool bare1 = !t->norm1, bare2 = !t->norm2;
+  if ((bare1 && (!t->post1 || sp->canon_taps > 0 || sp->norm_kind != 0 || sp->norm_offset != 0.f)) || (bare2 && sp->norm_kind != 0))
+    return fail(CAKE_B200_EINVAL, "layer %d: null norm1 needs post1, plain gains and no input convolution", layer_idx);
   const cake_b200_moe_spec &mo = sp->moe;
   const bool has_moe = mo.experts + mo.identity > 0;
   if (has_moe) {
-    if (sp->side || sp->canon_taps > 0 || sp->norm_offset != 0.f || sp->dense_ff > 0)
-      return fail(CAKE_B200_EINVAL, "layer %d: the routed feed-forward is not built beside a side mixer, an input convolution, offset gains or a dense feed-forward", layer_idx);
+    if (sp->canon_taps > 0 || sp->norm_offset != 0.f || sp->dense_ff > 0)
+      return fail(CAKE_B200_EINVAL, "layer %d: the routed feed-forward is not built beside an input convolution, offset gains or a dense feed-forward", layer_idx);
     if (mo.experts < 0 || mo.identity < 0 || mo.top < 1 || mo.top > mo.experts + mo.identity || mo.top > 32 || mo.experts + mo.identity > 256 ||
-        (mo.experts > 0 && mo.ff < 1) || mo.shared_ff < 0 || mo.act < 0 || mo.act > 2 || !t->norm2 || !t->router || !t->correction)
+        (mo.experts > 0 && mo.ff < 1) || mo.shared_ff < 0 || mo.act < 0 || mo.act > 3 || (bare2 && !t->post2) || !t->router || (mo.logit_bias && !t->correction) ||
+        (mo.groups > 1 && (mo.identity > 0 || mo.logit_bias || mo.experts % mo.groups || mo.groups_keep < 1 || mo.groups_keep > mo.groups ||
+                           mo.top > mo.groups_keep * (mo.experts / mo.groups))))
       return fail(CAKE_B200_EINVAL, "layer %d: bad router sizes (top <= 32, experts + identity <= 256) or null norm2 / router / correction", layer_idx);
     if (mo.experts > 0 && (!t->e_gate || !t->e_up || !t->e_down)) return fail(CAKE_B200_EINVAL, "layer %d: null expert table", layer_idx);
     if (mo.shared_ff > 0 && (!t->s_gate || !t->s_up || !t->s_down || !t->s_sg)) return fail(CAKE_B200_EINVAL, "layer %d: null shared-expert pointer", layer_idx);
@@ -2029,10 +2095,14 @@ static int load_mixer_ext(cake_b200_ctx *c, int layer_idx, const cake_b200_mixer
   }
   if (sp->side_dim < 0 || sp->side_col < 0 || (sp->side_dim > 0 && (!t->side_gate || !t->side_proj || !t->side_norm)))
     return fail(CAKE_B200_EINVAL, "layer %d: a token input needs side_gate / side_proj / side_norm", layer_idx);
-  if (sp->side && (!t->side || !t->branch_norm || !t->side->branch_norm)) return fail(CAKE_B200_EINVAL, "layer %d: a side mixer needs its tensors and both branch norms", layer_idx);
+  if (sp->side && (!t->side || !t->branch_norm != !t->side->branch_norm)) return fail(CAKE_B200_EINVAL, "layer %d: a side mixer needs its tensors and both branch norms or none", layer_idx);
+  const bool joint = sp->side && !t->branch_norm;  // added with constant factors: one output projection over both mixers' heads
+  auto scaled = [](int kind) { return kind == CAKE_B200_MIX_SINK_ATTENTION || kind == CAKE_B200_MIX_RETENTION; };
+  if (joint && (!scaled(sp->kind) || !scaled(sp->side->kind) || !t->o || !t->side->o))
+    return fail(CAKE_B200_EINVAL, "layer %d: mixers added with constant factors are built for sink attention and retention", layer_idx);
   if (sp->canon_taps < 0 || (sp->canon_taps > 0 && !t->canon)) return fail(CAKE_B200_EINVAL, "layer %d: canon_taps %d without canon", layer_idx, sp->canon_taps);
-  if (sp->dense_ff < 0 || (sp->dense_ff > 0 && (!t->ff_gate || !t->ff_up || !t->ff_down || !t->norm2 || sp->dense_act < 0 || sp->dense_act > 2)))
-    return fail(CAKE_B200_EINVAL, "layer %d: a dense feed-forward needs norm2 / ff_gate / ff_up / ff_down and dense_act in 0..2", layer_idx);
+  if (sp->dense_ff < 0 || (sp->dense_ff > 0 && (!t->ff_gate || !t->ff_up || !t->ff_down || (bare2 && !t->post2) || sp->dense_act < 0 || sp->dense_act > 3)))
+    return fail(CAKE_B200_EINVAL, "layer %d: a dense feed-forward needs norm2 / ff_gate / ff_up / ff_down and dense_act in 0..3", layer_idx);
   CU(cudaSetDevice(c->device));
   const size_t es = c->es, H = c->cfg.hidden;
   auto *b = new cake_b200_block{c, layer_idx, c->device};
@@ -2041,11 +2111,20 @@ static int load_mixer_ext(cake_b200_ctx *c, int layer_idx, const cake_b200_mixer
   const int rc = [&]() -> int {
     std::vector<InPart> parts;
     size_t row = 0;
-    RC(load_sub_mixer(c, b, sp, t, parts, row, layer_idx));
+    RC(load_sub_mixer(c, b, sp, t, parts, row, layer_idx, joint));
     if (sp->side) {
       b->side = new cake_b200_block{c, layer_idx, c->device};
       b->side->mixer = b->side->ext = true;
-      RC(load_sub_mixer(c, b->side, sp->side, t->side, parts, row, layer_idx));
+      RC(load_sub_mixer(c, b->side, sp->side, t->side, parts, row, layer_idx, joint));
+    }
+    if (joint) {  // the factors go onto the heads in fp32, before they are rounded to D
+      const size_t ia = (size_t)sp->heads * sp->vdim, ib = (size_t)sp->side->heads * sp->side->vdim;
+      b->joint = true;
+      b->out_scale = sp->branch_scale;
+      b->side->out_scale = sp->side->branch_scale;
+      CU(cudaMalloc(&b->wo, H * (ia + ib) * es + 16));
+      RC(pipe_copy(c, b->wo, (ia + ib) * es, t->o, ia * es, ia * es, H));
+      RC(pipe_copy(c, (char *)b->wo + ia * es, (ia + ib) * es, t->side->o, ib * es, ib * es, H));
     }
     // block-level switches live in the main block's spec
     b->ms.norm_offset = sp->norm_offset;
@@ -2075,12 +2154,12 @@ static int load_mixer_ext(cake_b200_ctx *c, int layer_idx, const cake_b200_mixer
       if (pr.bias) RC(pipe_copy(c, (char *)b->b_in + r * es, pr.rows * es, pr.bias, pr.rows * es, pr.rows * es, 1));
       r += pr.rows;
     }
-    RC(upload(c, &b->ln1, t->norm1, H * es));
+    if (t->norm1) RC(upload(c, &b->ln1, t->norm1, H * es));
     if (t->post1) RC(upload(c, &b->post1, t->post1, H * es));
     if (sp->canon_taps > 0) RC(upload(c, &b->canon, t->canon, H * sp->canon_taps * es));
     if (sp->dense_ff > 0) {  // row-interleaved gate / up as everywhere else
       const size_t I = sp->dense_ff;
-      RC(upload(c, &b->ln2, t->norm2, H * es));
+      if (t->norm2) RC(upload(c, &b->ln2, t->norm2, H * es));
       if (t->post2) RC(upload(c, &b->post2, t->post2, H * es));
       CU(cudaMalloc(&b->wgu, 2 * I * H * es + 16));
       RC(pipe_copy(c, b->wgu, 2 * H * es, t->ff_gate, H * es, H * es, I));
@@ -2139,6 +2218,11 @@ static int cache_ensure_sub(cake_b200_cache *k, int slot, const cake_b200_block 
   if (kv_rows) {
     CU(cudaMalloc(&k->k[slot], (size_t)k->batch * G * k->cap * sp.dim * c->es + 16));
     CU(cudaMalloc(&k->v[slot], (size_t)k->batch * G * k->cap * sp.vdim * c->es + 16));
+    if (sp.kind == CAKE_B200_MIX_SINK_ATTENTION && sp.pool > 0) {  // one row per complete block, beside the rows it stands for
+      const size_t rows = (size_t)k->batch * G * std::max(1, k->cap / sp.pool);
+      CU(cudaMalloc(&k->pk[slot], rows * sp.dim * c->es + 16));
+      CU(cudaMalloc(&k->pv[slot], rows * sp.vdim * c->es + 16));
+    }
     if (talk_on_tc(c, b)) CU(cudaMalloc(&k->vt[slot], (size_t)k->batch * G * sp.vdim * latent_cap_t(k->cap) * c->es + 16));
   } else if (sp.kind == CAKE_B200_MIX_LATENT_WINDOW) {  // the normed latent: one row per position for all heads
     CU(cudaMalloc(&k->k[slot], (size_t)k->batch * k->cap * sp.kv_rank * c->es + 16));
@@ -2180,15 +2264,17 @@ static bool window_on_tc(const cake_b200_ctx *c, const cake_b200_block *b, int S
   }();
   const cake_b200_mixer_spec &sp = b->ms;
   if (off || c->cfg.dtype == CAKE_B200_F32 || S < WIN_TC_MIN_ROWS || sp.dim != FT_HD || sp.vdim != FT_HD || b->n_in_pad % 8 != 0) return false;
+  if (b->joint && (b->side->ms.heads * b->side->ms.vdim) % 8 != 0) return false;  // the output rows of both mixers are 16-byte pieces
   if (sp.kind == CAKE_B200_MIX_SINK_ATTENTION) return b->pc[3] < 0 || b->pc[3] % 8 == 0;
   return sp.kind == CAKE_B200_MIX_LATENT_WINDOW && sp.kv_rank % TC_BK == 0;
 }
-template <typename Take> static SubScratch sub_scratch(const cake_b200_ctx *c, const cake_b200_block *b, size_t M, int S, int n_keys, Take &&take) {
+// att_cols: columns of the heads' output (0: the caller shares the other mixer's buffers)
+template <typename Take> static SubScratch sub_scratch(const cake_b200_ctx *c, const cake_b200_block *b, size_t M, int S, int n_keys, size_t att_cols, Take &&take) {
   SubScratch s{};
   const cake_b200_mixer_spec &sp = b->ms;
   const size_t es = c->es, inner = (size_t)sp.heads * sp.vdim, G = sp.kv_heads;
-  s.att = take(M * inner * es);
-  s.y = (float *)take(M * c->cfg.hidden * sizeof(float));
+  if (att_cols) s.att = take(M * att_cols * es);
+  if (att_cols) s.y = (float *)take(M * c->cfg.hidden * sizeof(float));
   if (sp.kind == CAKE_B200_MIX_SINK_ATTENTION || sp.kind == CAKE_B200_MIX_LATENT_WINDOW) {
     const bool latent = sp.kind == CAKE_B200_MIX_LATENT_WINDOW;
     const size_t vd = latent ? sp.kv_rank : sp.vdim;
@@ -2205,7 +2291,9 @@ template <typename Take> static SubScratch sub_scratch(const cake_b200_ctx *c, c
       }
     }
     // steps of a few rows over many visible keys: split the keys so that the step fills the chip
-    const int vis = std::min(n_keys, sp.window > 0 ? sp.window + sp.keep_first : n_keys);
+    int vis = std::min(n_keys, sp.window > 0 ? sp.window + sp.keep_first : n_keys);
+    if (sp.chunk > 0) vis = std::min(vis, sp.chunk);
+    if (sp.pool > 0 && n_keys > sp.window) vis += (n_keys - sp.window) / sp.pool;
     if (M * sp.heads <= 1024 && vis >= 256) {
       s.nsplit = (int)std::min<size_t>(WIN_SPLIT_MAX, std::min<size_t>((vis + 63) / 64, (2 * (size_t)c->sm_count + M * sp.heads - 1) / (M * sp.heads)));
       if (s.nsplit > 1) s.part = (float *)take(M * sp.heads * s.nsplit * (vd + 2) * sizeof(float));
@@ -2237,6 +2325,7 @@ template <typename Take> static SubScratch sub_scratch(const cake_b200_ctx *c, c
     return s;
   }
   s.o32 = (float *)take(M * inner * sizeof(float));
+  if (sp.kind == CAKE_B200_MIX_RETENTION) return s;
   s.f1 = (float *)take(M * sp.heads * sizeof(float));
   s.f2 = (float *)take(M * sp.heads * sizeof(float));
   if (sp.kind == CAKE_B200_MIX_DELTA) {
@@ -2275,8 +2364,10 @@ static ExtScratch ext_scratch(const cake_b200_ctx *c, const cake_b200_block *b, 
   s.h = take(M * H * es);
   if (b->ms.canon_taps > 0) s.h32 = (float *)take(M * H * sizeof(float));
   s.proj = take(M * b->n_in_pad * es);
-  s.a = sub_scratch(c, b, M, S, n_keys, take);
-  if (b->side) s.b = sub_scratch(c, b->side, M, S, n_keys, take);
+  const size_t ia = (size_t)b->ms.heads * b->ms.vdim, ib = b->side ? (size_t)b->side->ms.heads * b->side->ms.vdim : 0;
+  s.a = sub_scratch(c, b, M, S, n_keys, b->joint ? ia + ib : ia, take);
+  if (b->side) s.b = sub_scratch(c, b->side, M, S, n_keys, b->joint ? 0 : ib, take);
+  if (b->joint) s.b.att = base ? (char *)s.a.att + ia * es : nullptr;
   if (b->ms.dense_ff > 0) s.act = take(M * (size_t)b->ms.dense_ff * es);
   if (b->ms.side_dim > 0) s.side = take(M * (size_t)b->ms.side_dim * es);
   s.moe = moe_scratch(c, b, M, take);
@@ -2298,9 +2389,10 @@ template <> int gemm_bias_tc<float>(cake_b200_ctx *, const void *, const void *,
 // one mixer of an ext block: proj [M, ldp] holds its projections at b->pc[]; y [M, hidden] fp32 receives o(att) without o's bias
 template <typename T>
 static int run_sub_mixer(cake_b200_ctx *c, const cake_b200_block *b, cake_b200_cache *kc, int slot, const SubScratch &w, const T *proj, int ldp,
-                         int B, int S, int pos0, uint64_t *lc, cudaStream_t st, bool with_out) {
+                         int B, int S, int pos0, uint64_t *lc, cudaStream_t st, bool with_out, int ld_att = 0) {
   const cake_b200_mixer_spec &sp = b->ms;
   const int M = B * S, H = c->cfg.hidden, dt = c->cfg.dtype, G = sp.kv_heads, inner = sp.heads * sp.vdim;
+  const int ldo = ld_att ? ld_att : inner;  // row stride of the heads' output (both mixers side by side in a joint block)
   if (sp.kind == CAKE_B200_MIX_DELTA) {
     const int qk = G * sp.dim, ch = 2 * qk + inner;
     const T *cv = (const T *)w.conv;
@@ -2352,17 +2444,29 @@ static int run_sub_mixer(cake_b200_ctx *c, const cake_b200_block *b, cake_b200_c
     }
   } else if (sp.kind == CAKE_B200_MIX_SINK_ATTENTION) {
     mx::QkPrep qp{proj, ldp, b->pc[0], b->pc[1], b->pc[2], b->m_cos, b->m_sin, sp.rot.dims, sp.qk_unit, c->cfg.rms_eps, w.qh, kc->k[slot], kc->v[slot],
-                  B, S, sp.heads, G, sp.dim, sp.vdim, kc->cap, pos0};
+                  B, S, sp.heads, G, sp.dim, sp.vdim, kc->cap, pos0, sp.rot.interleaved, b->m_qn, b->m_kn, sp.v_unit};
     MX(mx::qk_prep(st, dt, qp, lc));
-    mx::WindowAttn wa{w.qh, sp.heads * sp.dim, kc->k[slot], kc->v[slot], b->pc[3] >= 0 ? proj + b->pc[3] : nullptr, ldp, 0, b->m_sink, w.att, inner,
-                      B, S, sp.heads, G, sp.dim, sp.vdim, kc->cap, pos0, sp.window, sp.keep_first, sp.scale, w.part, w.nsplit};
+    const int pcap = sp.pool > 0 ? std::max(1, kc->cap / sp.pool) : 0;
+    if (sp.pool > 0) {  // the blocks that this step completes
+      mx::PoolRows pr{kc->k[slot], kc->v[slot], kc->pk[slot], kc->pv[slot], B, S, G, sp.dim, sp.vdim, kc->cap, pcap, pos0, sp.pool};
+      MX(mx::pool_rows(st, dt, pr, lc));
+    }
+    mx::WindowAttn wa{w.qh, sp.heads * sp.dim, kc->k[slot], kc->v[slot], b->pc[3] >= 0 ? proj + b->pc[3] : nullptr, ldp, 0, b->m_sink, w.att, ldo,
+                      B, S, sp.heads, G, sp.dim, sp.vdim, kc->cap, pos0, sp.window, sp.keep_first, sp.scale, w.part, w.nsplit,
+                      kc->pk[slot], kc->pv[slot], sp.pool, pcap, sp.chunk, sp.sink_zero, sp.softcap, b->out_scale};
     if (window_on_tc(c, b, S)) {
       const void *gate = b->pc[3] >= 0 ? proj + b->pc[3] : nullptr;
-      WinAttn ta{w.qh, kc->k[slot], kc->v[slot], nullptr, nullptr, w.att, B, S, sp.heads, G, FT_HD, kc->cap, pos0, sp.heads * FT_HD, inner, -1, sp.window,
-                 sp.scale, 0.f, sp.keep_first, 0, b->m_sink, gate, gate ? 2 : 0, ldp};
-      RC(window_attention_tc<T>(c, ta, 0, lc));
+      WinAttn ta{w.qh, kc->k[slot], kc->v[slot], nullptr, nullptr, w.att, B, S, sp.heads, G, FT_HD, kc->cap, pos0, sp.heads * FT_HD, ldo, -1, sp.window,
+                 sp.scale, sp.softcap, sp.keep_first, 0, b->m_sink, gate, gate ? 2 : 0, ldp, sp.pool, sp.chunk, sp.sink_zero, b->out_scale};
+      RC(window_attention_tc<T>(c, ta, 0, lc, kc->pk[slot], kc->pv[slot], pcap));
     } else if (mx::window_attention_tiled_ok(dt, wa)) MX(mx::window_attention_tiled(st, dt, wa, lc));
     else MX(mx::window_attention(st, dt, wa, lc));
+  } else if (sp.kind == CAKE_B200_MIX_RETENTION) {
+    mx::Recurrence r{proj + b->pc[0], proj + b->pc[1], proj + b->pc[2], ldp, ldp, ldp, 1, nullptr, 0, nullptr, nullptr, nullptr, b->m_decay,
+                     1.0f / sqrtf((float)sp.dim), b->m_cos, b->m_sin, sp.rot.dims, kc->rec_state[slot], w.o32, B, S, sp.heads, sp.dim, sp.vdim, pos0};
+    MX(mx::recurrence(st, dt, r, lc));
+    mx::GateNorm gn{w.o32, proj + b->pc[3], ldp, nullptr, w.att, M, inner, sp.heads, 0, c->cfg.rms_eps, 0, 0, nullptr, ldo, b->out_scale};
+    MX(mx::gate_norm(st, dt, gn, lc));
   } else if (sp.kind == CAKE_B200_MIX_LATENT_WINDOW) {
     // both latents are normed (the key / value latent straight into the cache), the query latent is expanded and taken through
     // the key expansion, so that the attention runs over the cached latent rows for all heads: qa_h = uk_h^T q_h,
@@ -2415,9 +2519,11 @@ static int run_sub_mixer(cake_b200_ctx *c, const cake_b200_block *b, cake_b200_c
 }
 
 // one ext block: x_out = x + post1(mixers(canon(norm1(x)))), then x_out += post2(ff(norm2(x_out)))
+// Blocks without norms in front of their sublayers read the stream rounded to D (D = float: the stream as it stands): the kernel
+// that adds a sublayer's output leaves it in the scratch's first buffer, which every block of a step shares; x_in_h: it is there.
 template <typename T>
 static int enqueue_ext_layer(cake_b200_ctx *c, const cake_b200_block *b, int l, cake_b200_cache *kc, const float *cur, float *x_out, int B, int S, int pos0,
-                             uint64_t *lc) {
+                             uint64_t *lc, bool &x_in_h) {
   const cake_b200_mixer_spec &sp = b->ms;
   const int M = B * S, H = c->cfg.hidden, dt = c->cfg.dtype, nl = (int)kc->len.size();
   const float eps = c->cfg.rms_eps;
@@ -2425,7 +2531,18 @@ static int enqueue_ext_layer(cake_b200_ctx *c, const cake_b200_block *b, int l, 
   const ExtScratch w = ext_scratch(c, b, (size_t)M, (char *)c->mx_ws, S, pos0 + S);
   // 1. h = norm1(x), the input convolution, every projection of the mixer(s) in one product
   const bool squash = sp.norm_kind == 1;  // tanh(alpha x) * w + b instead of an RMS norm, in all four places
-  if (squash) {
+  const bool wide = dt == CAKE_B200_F32;
+  auto stream_operand = [&](const float *x) -> const void * {
+    if (wide) return x;
+    if (!x_in_h && mx::rows_to_d(st, dt, x, w.h, (size_t)M * H, lc) != 0) return nullptr;
+    return w.h;
+  };
+  const void *op = w.h;
+  if (b->ln1) x_in_h = false;
+  if (!b->ln1) {
+    op = stream_operand(cur);
+    if (!op) return fail(CAKE_B200_ECUDA, "rounding the stream: %s", cudaGetErrorString(cudaGetLastError()));
+  } else if (squash) {
     mx::TanhNorm n1{cur, nullptr, 1, 0, b->ln1, b->ln1_b, sp.norm_alpha[0], nullptr, nullptr, w.h, M, H};
     MX(mx::tanh_norm(st, dt, n1, lc));
   } else {
@@ -2436,13 +2553,14 @@ static int enqueue_ext_layer(cake_b200_ctx *c, const cake_b200_block *b, int l, 
     mx::CanonConv cc{w.h32, b->canon, kc->canon_hist[l], w.h, B, S, H, sp.canon_taps, pos0};
     MX(mx::canon_conv(st, dt, cc, lc));
   }
-  if (listed_tc<T>(c, M, b->n_in_pad, H)) RC(gemm_bias_tc<T>(c, w.h, b->w_in, b->b_in, w.proj, M, b->n_in_pad, H));
+  if (listed_tc<T>(c, M, b->n_in_pad, H)) RC(gemm_bias_tc<T>(c, op, b->w_in, b->b_in, w.proj, M, b->n_in_pad, H));
   else {
-    RowsGemm gi{w.h, b->w_in, nullptr, w.proj, M, b->n_in, H, H, b->n_in_pad, 0, 0.f, nullptr, b->b_in};
+    RowsGemm gi{op, b->w_in, nullptr, w.proj, M, b->n_in, H, H, b->n_in_pad, 0, 0.f, nullptr, b->b_in};
     RC((gemm_rows_T<T, RE_STORE>(c, gi)));
   }
   // 2. the mixer(s), each up to its output projection in fp32
   // a recurrent side mixer (its kernels take a stream; its few CTAs leave most of the chip idle) runs next to the main mixer
+  const int ld_att = b->joint ? sp.heads * sp.vdim + b->side->ms.heads * b->side->ms.vdim : 0;
   const bool fork = b->side && b->side->ms.kind != CAKE_B200_MIX_TALKING_ATTENTION && M >= 256 && !c->capturing;
   if (fork) {
     if (!c->side_stream) {
@@ -2452,16 +2570,33 @@ static int enqueue_ext_layer(cake_b200_ctx *c, const cake_b200_block *b, int l, 
     }
     CU(cudaEventRecord(c->ev_fork, st));
     CU(cudaStreamWaitEvent(c->side_stream, c->ev_fork, 0));
-    RC(run_sub_mixer<T>(c, b->side, kc, nl + l, w.b, (const T *)w.proj, b->n_in_pad, B, S, pos0, lc, c->side_stream, false));
+    RC(run_sub_mixer<T>(c, b->side, kc, nl + l, w.b, (const T *)w.proj, b->n_in_pad, B, S, pos0, lc, c->side_stream, false, ld_att));
     CU(cudaEventRecord(c->ev_join, c->side_stream));
   }
-  RC(run_sub_mixer<T>(c, b, kc, l, w.a, (const T *)w.proj, b->n_in_pad, B, S, pos0, lc, st, true));
-  if (fork) {
+  RC(run_sub_mixer<T>(c, b, kc, l, w.a, (const T *)w.proj, b->n_in_pad, B, S, pos0, lc, st, !b->joint, ld_att));
+  if (b->joint) {
+    if (fork) CU(cudaStreamWaitEvent(st, c->ev_join, 0));
+    else RC(run_sub_mixer<T>(c, b->side, kc, nl + l, w.b, (const T *)w.proj, b->n_in_pad, B, S, pos0, lc, st, false, ld_att));
+    RC(gemm_f32_out<T>(c, w.a.att, b->wo, w.a.y, M, H, ld_att));
+  } else if (fork) {
     CU(cudaStreamWaitEvent(st, c->ev_join, 0));
     RC(gemm_f32_out<T>(c, w.b.att, b->side->wo, w.b.y, M, H, b->side->ms.heads * b->side->ms.vdim));
   } else if (b->side) RC(run_sub_mixer<T>(c, b->side, kc, nl + l, w.b, (const T *)w.proj, b->n_in_pad, B, S, pos0, lc, st, true));
   // 3. x <- x + post1(branches)
-  if (squash && b->post1) {
+  const bool has_moe = sp.moe.experts + sp.moe.identity > 0;
+  // a sublayer that is normed on its output only: norm, residual sum and the next sublayer's operand in one pass
+  const bool bare_ff = !b->ln2 && (sp.dense_ff > 0 || has_moe);
+  auto merge = [&](const float *a, const void *post, const float *x, const MoeScratch *mo) -> int {
+    mx::StreamMerge sm{mo ? nullptr : a, mo ? mo->y : nullptr, mo ? mo->wts : nullptr, mo ? mo->ids : nullptr, mo ? mo->pos_of : nullptr,
+                       mo ? sp.moe.top : 0, mo ? sp.moe.experts : 0, post, x, x_out, wide ? nullptr : w.h, M, H, eps};
+    MX(mx::stream_merge(st, dt, sm, lc));
+    x_in_h = !wide;
+    return CAKE_B200_OK;
+  };
+  x_in_h = false;
+  if (!b->ln1 && (!b->side || b->joint) && !b->m_ob) {
+    RC(merge(w.a.y, b->post1, cur, nullptr));
+  } else if (squash && b->post1) {
     mx::TanhNorm p1{w.a.y, nullptr, 1, 0, b->post1, b->post1_b, sp.norm_alpha[1], cur, x_out, nullptr, M, H};
     MX(mx::tanh_norm(st, dt, p1, lc));
   } else {
@@ -2470,8 +2605,12 @@ static int enqueue_ext_layer(cake_b200_ctx *c, const cake_b200_block *b, int l, 
     MX(mx::branch_merge(st, dt, bm, lc));
   }
   // 4. x <- x + post2(ff(norm2(x)))
-  const bool has_moe = sp.moe.experts + sp.moe.identity > 0;
-  if (sp.dense_ff > 0 || has_moe) {
+  op = w.h;
+  if (bare_ff) {
+    op = stream_operand(x_out);
+    if (!op) return fail(CAKE_B200_ECUDA, "rounding the stream: %s", cudaGetErrorString(cudaGetLastError()));
+  } else if (sp.dense_ff > 0 || has_moe) {
+    x_in_h = false;
     if (squash) {
       mx::TanhNorm n2{x_out, nullptr, 1, 0, b->ln2, b->ln2_b, sp.norm_alpha[2], nullptr, nullptr, w.h, M, H};
       MX(mx::tanh_norm(st, dt, n2, lc));
@@ -2481,8 +2620,12 @@ static int enqueue_ext_layer(cake_b200_ctx *c, const cake_b200_block *b, int l, 
     }
   }
   if (has_moe) {  // the feed-forward's sum lands in y; a post norm squashes it on its way into the stream
-    if (b->post2) {
-      RC(enqueue_routed_ff<T>(c, b, w.moe, w.h, nullptr, w.a.y, M, lc));
+    if (bare_ff && b->post2 && sp.moe.identity == 0 && !sp.moe.shared_ff) {  // the experts' outputs are summed by the kernel that norms the sum
+      RC(enqueue_routed_ff<T>(c, b, w.moe, op, nullptr, nullptr, M, lc));
+      RC(merge(nullptr, b->post2, x_out, &w.moe));
+    } else if (b->post2) {
+      RC(enqueue_routed_ff<T>(c, b, w.moe, op, nullptr, w.a.y, M, lc));
+      x_in_h = false;
       if (squash) {
         mx::TanhNorm p2{w.a.y, nullptr, 1, 0, b->post2, b->post2_b, sp.norm_alpha[3], x_out, x_out, nullptr, M, H};
         MX(mx::tanh_norm(st, dt, p2, lc));
@@ -2490,17 +2633,18 @@ static int enqueue_ext_layer(cake_b200_ctx *c, const cake_b200_block *b, int l, 
         mx::BranchMerge fm{w.a.y, nullptr, nullptr, nullptr, nullptr, nullptr, b->post2, sp.norm_offset, x_out, x_out, M, H, eps};
         MX(mx::branch_merge(st, dt, fm, lc));
       }
-    } else RC(enqueue_routed_ff<T>(c, b, w.moe, w.h, x_out, x_out, M, lc));
+    } else RC(enqueue_routed_ff<T>(c, b, w.moe, op, x_out, x_out, M, lc));
   }
   if (sp.dense_ff > 0) {
     const int I = sp.dense_ff;
-    if (listed_tc<T>(c, M, 2 * I, H)) RC((listed_gemm_tc<T, TCE_SWIGLU>(c, w.h, b->wgu, nullptr, w.act, M, 2 * I, H, sp.dense_act, I, sp.dense_limit)));
+    if (listed_tc<T>(c, M, 2 * I, H)) RC((listed_gemm_tc<T, TCE_SWIGLU>(c, op, b->wgu, nullptr, w.act, M, 2 * I, H, sp.dense_act, I, sp.dense_limit)));
     else {
-      RowsGemm gu{w.h, b->wgu, nullptr, w.act, M, 2 * I, H, H, I, sp.dense_act, sp.dense_limit};
+      RowsGemm gu{op, b->wgu, nullptr, w.act, M, 2 * I, H, H, I, sp.dense_act, sp.dense_limit};
       RC((gemm_rows_T<T, RE_GATE_UP>(c, gu)));
     }
     RC(gemm_f32_out<T>(c, w.act, b->wd, w.a.y, M, H, I));
-    if (squash && b->post2) {
+    if (bare_ff) RC(merge(w.a.y, b->post2, x_out, nullptr));
+    else if (squash && b->post2) {
       mx::TanhNorm p2{w.a.y, nullptr, 1, 0, b->post2, b->post2_b, sp.norm_alpha[3], x_out, x_out, nullptr, M, H};
       MX(mx::tanh_norm(st, dt, p2, lc));
     } else {
@@ -2510,6 +2654,7 @@ static int enqueue_ext_layer(cake_b200_ctx *c, const cake_b200_block *b, int l, 
   }
   // 5. the per-layer token input
   if (sp.side_dim > 0) {
+    x_in_h = false;
     if (!c->side_tab || sp.side_col + sp.side_dim > c->side_cols) return fail(CAKE_B200_ESTATE, "layer %d: the token input needs columns %d..%d of the side table (%d loaded)", b->layer, sp.side_col, sp.side_col + sp.side_dim, c->side_cols);
     if (c->d_ids_n != (size_t)M) return fail(CAKE_B200_ESTATE, "layer %d: the token input needs the ids of this step (%zu embedded, %d rows)", b->layer, c->d_ids_n, M);
     // g = gelu(G x) * e and y = P g as two products with the gate between them; x += rms(y) * w is a merge with a post norm
@@ -2642,7 +2787,7 @@ static int enqueue_routed_ff(cake_b200_ctx *c, const cake_b200_block *b, const M
   if (listed_tc<T>(c, M, NP, H)) RC((listed_gemm_tc<T, TCE_SOFTCAP_F32>(c, h, b->m_router, nullptr, w.logits, M, NP, H, 0, 0)));
   else RC((gemm_rows_T<T, RE_SOFTCAP_F32>(c, gr)));
   mx::MoePlan mp{w.logits, NP, b->m_corr, mo.shared_ff ? 1 : 0, M, H, mo.experts, mo.identity, mo.top, mo.scale, w.ids, w.wts,
-                 w.sgate, w.tile, w.counts, w.perm, w.pos_of, w.tile_expert, w.max_tiles, mo.logit_bias};
+                 w.sgate, w.tile, w.counts, w.perm, w.pos_of, w.tile_expert, w.max_tiles, mo.logit_bias, mo.groups, mo.groups_keep, mo.plain_weights};
   MX(mx::moe_route(st, dt, mp, lc));
   if (mo.experts && w.sorted) {  // grouped products: sorted rows of h -> act(gate) * up -> down, expert e at row e * N of the stacked weights
     const int rows = w.max_tiles * w.tile;
@@ -2656,6 +2801,7 @@ static int enqueue_routed_ff(cake_b200_ctx *c, const cake_b200_block *b, const M
     mx::MoeExperts me{h, b->m_eg, b->m_ed, w.act, w.y, M, H, mo.ff, mo.top, mo.act, w.perm, w.tile_expert, w.tile, w.max_tiles, mo.limit};
     MX(mx::moe_experts(st, dt, me, lc));
   }
+  if (!out) return CAKE_B200_OK;  // the caller sums the sorted outputs itself
   mx::MoeCombine mc{x, out, h, w.y, w.wts, w.ids, w.pos_of, M, H, mo.top, mo.experts};
   MX(mx::moe_combine(st, dt, mc, lc));
   if (mo.shared_ff) {
@@ -2680,7 +2826,8 @@ static int enqueue_mixer_layers(cake_b200_ctx *c, cake_b200_block *const *blocks
   for (int i = 0; i < n; i++) {
     need = std::max(need, blocks[i]->ext ? ext_scratch(c, blocks[i], (size_t)M, nullptr, S, pos0 + S).total
                                          : mixer_scratch(c, blocks[i], (size_t)M, nullptr, S, pos0 + S).total);
-    if (blocks[i]->m_cos && pos0 + S > blocks[i]->m_rope_rows)
+    const cake_b200_block *sd = blocks[i]->side;
+    if ((blocks[i]->m_cos && pos0 + S > blocks[i]->m_rope_rows) || (sd && sd->m_cos && pos0 + S > sd->m_rope_rows))
       return fail(CAKE_B200_ESTATE, "position %d exceeds the rotation table (%d rows = the ctx's max_seq)", pos0 + S, blocks[i]->m_rope_rows);
   }
   if (need > c->mx_ws_cap) {
@@ -2696,15 +2843,17 @@ static int enqueue_mixer_layers(cake_b200_ctx *c, cake_b200_block *const *blocks
   return DISPATCH_T3(dt, T_LAMBDA {
     typedef typename decltype(tag_)::type T;
     const float *cur = x_in;
+    bool x_in_h = false;
     for (int i = 0; i < n; i++) {
       const cake_b200_block *b = blocks[i];
       const cake_b200_mixer_spec &sp = b->ms;
       const int l = block_idx[i], inner = sp.heads * sp.vdim;
       if (b->ext) {
-        RC(enqueue_ext_layer<T>(c, b, l, kc, cur, x_out, B, S, pos0, lc));
+        RC(enqueue_ext_layer<T>(c, b, l, kc, cur, x_out, B, S, pos0, lc, x_in_h));
         cur = x_out;
         continue;
       }
+      x_in_h = false;
       const MixerScratch w = mixer_scratch(c, b, (size_t)M, (char *)c->mx_ws, S, pos0 + S);
       // 1. h = norm1(x); every input projection of the mixer in one product
       RC(launch_pdl(c, norm_shift_rows_kernel<T>, dim3(M), dim3(256), 0, cur, (const int *)nullptr, 1, 0, (const T *)b->ln1, 1, (const T *)nullptr,
@@ -2968,6 +3117,11 @@ extern "C" int cake_b200_embed(cake_b200_ctx *c, const uint32_t *ids_host, int b
   CU(cudaMemcpyAsync(c->d_ids, ids_host, n * 4, cudaMemcpyHostToDevice, c->stream));
   c->d_ids_n = n;
   // the ids buffer is pageable in general: the copy above returns after staging, safe to reuse
+  if (c->embed_norm) {
+    MX(mx::embed_norm(c->stream, c->cfg.dtype, c->embed, c->d_ids, c->embed_norm, (float *)x_dev, (int)n, c->cfg.hidden, c->cfg.vocab, c->cfg.embed_scale,
+                      c->cfg.rms_eps, &c->launches));
+    return CAKE_B200_OK;
+  }
   if (c->cfg.layer_list)  // the fp32 residual stream starts here
     return DISPATCH_T3(c->cfg.dtype, T_LAMBDA {
       typedef typename decltype(tag_)::type T;
@@ -3000,6 +3154,10 @@ extern "C" int cake_b200_head_load_tables(cake_b200_ctx *c, const cake_b200_embe
     c->pos_rows = t->pos_rows;
   }
   c->final_norm_offset = t->final_norm_offset;
+  if (t->embed_norm) {
+    if (t->bigram || t->pos) return fail(CAKE_B200_EINVAL, "the norm behind the embedding is not built beside pair or position tables");
+    RC(upload(c, &c->embed_norm, t->embed_norm, H * c->es));
+  }
   if (t->side) {
     if (t->side_cols < 1) return fail(CAKE_B200_EINVAL, "bad side table size");
     RC(upload(c, &c->side_tab, t->side, (size_t)c->cfg.vocab * t->side_cols * c->es));

@@ -63,7 +63,7 @@ template <typename T> __device__ __forceinline__ float gate_act(float g, int act
 }
 
 // act(gate) * up of a gated feed-forward from the two fp32 accumulators.  act 0 / 1: as gate_act.  act 2, the clamped form:
-// g' = min(g, lim), u' = clamp(u, -lim, lim), g' * sigmoid(1.702 g') * (u' + 1).
+// g' = min(g, lim), u' = clamp(u, -lim, lim), g' * sigmoid(1.702 g') * (u' + 1).  act 3: max(g, 0) * u.
 template <typename T> __device__ __forceinline__ float gated_pair(float g, float u, int act, float lim) {
   g = rnd<T>(g);
   u = rnd<T>(u);
@@ -72,6 +72,7 @@ template <typename T> __device__ __forceinline__ float gated_pair(float g, float
     u = fminf(fmaxf(u, -lim), lim);
     return g / (1.0f + expf(-1.702f * g)) * (u + 1.0f);
   }
+  if (act == 3) return fmaxf(g, 0.f) * u;
   return gate_act<T>(g, act) * u;
 }
 

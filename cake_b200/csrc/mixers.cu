@@ -817,14 +817,14 @@ __global__ void __launch_bounds__(128) gate_norm_kernel(const GateNorm p) {
   const float *o = p.o + (size_t)m * p.n + c0;
   const T *gate = reinterpret_cast<const T *>(p.gate) + (size_t)m * p.ldg + c0;
   const T *w = p.w ? reinterpret_cast<const T *>(p.w) + (p.w_period ? 0 : c0) : nullptr;  // w_period == len: every part reads the same gains
-  T *out = reinterpret_cast<T *>(p.out) + (size_t)m * p.n + c0;
+  T *out = reinterpret_cast<T *>(p.out) + (size_t)m * (p.ldo ? p.ldo : p.n) + c0;
   const float rdiv = p.row_div ? p.row_div[(size_t)m * p.parts + g] : 1.f;
   const bool sg = p.gate_sigmoid != 0;
   auto gact = [sg](float z) { return sg ? 1.0f / (1.0f + expf(-z)) : silu_f(z); };
   float ss = 0.f;
   // parts whose rows start on 16 bytes: four entries per lane and load
-  const bool vec = sizeof(T) == 2 && (len & 3) == 0 && (p.n & 3) == 0 && (p.ldg & 3) == 0 &&
-                   (((uintptr_t)p.o | (uintptr_t)p.out) & 15) == 0 && (((uintptr_t)p.gate | (uintptr_t)(p.w ? p.w : p.gate)) & 7) == 0;
+  const bool vec = sizeof(T) == 2 && (len & 3) == 0 && (p.n & 3) == 0 && (p.ldg & 3) == 0 && (p.ldo & 3) == 0 &&
+                   ((uintptr_t)p.o & 15) == 0 && ((uintptr_t)p.out & 7) == 0 && (((uintptr_t)p.gate | (uintptr_t)(p.w ? p.w : p.gate)) & 7) == 0;
   if (vec) {
     const float4 *o4 = reinterpret_cast<const float4 *>(o);
     const uint2 *g2 = reinterpret_cast<const uint2 *>(gate), *w2 = reinterpret_cast<const uint2 *>(w);
@@ -860,7 +860,7 @@ __global__ void __launch_bounds__(128) gate_norm_kernel(const GateNorm p) {
         float r = (p.gate_first ? v[e] * gs[e] : v[e]) * inv;
         if (w) r *= wv[e];
         if (!p.gate_first) r *= gs[e];
-        v[e] = r;
+        v[e] = r * p.out_scale;
       }
       *reinterpret_cast<uint2 *>(out + 4 * i) = make_uint2(pack2x<B>(v[0], v[1]), pack2x<B>(v[2], v[3]));
     }
@@ -879,7 +879,7 @@ __global__ void __launch_bounds__(128) gate_norm_kernel(const GateNorm p) {
     float v = (p.gate_first ? ov * gs : ov) * inv;
     if (w) v *= DT<T>::to_f(w[i]);
     if (!p.gate_first) v *= gs;
-    out[i] = DT<T>::from_f(v);
+    out[i] = DT<T>::from_f(v * p.out_scale);
   }
 }
 int gate_norm(cudaStream_t st, int dtype, const GateNorm &p, uint64_t *launches) {
@@ -923,7 +923,47 @@ __global__ void __launch_bounds__(128) moe_router_kernel(const MoePlan p) {
       continue;
     }
     sc[sI] = sc[sI] / sum;
-    ch[sI] = e < E ? sc[sI] + DT<T>::to_f(corr[e]) : -INFINITY;
+    ch[sI] = e < E ? sc[sI] + (corr ? DT<T>::to_f(corr[e]) : 0.f) : -INFINITY;
+  }
+  if (p.groups > 1) {  // lane g keeps the best score of group g (g = lane + 32 sI); the best groups_keep groups stay open
+    const int gsz = E / p.groups;
+    float gb[MOE_MAX_SLOTS];
+    bool open[MOE_MAX_SLOTS];
+#pragma unroll
+    for (int sI = 0; sI < MOE_MAX_SLOTS; sI++) { gb[sI] = -INFINITY; open[sI] = false; }
+    for (int g = 0; g < p.groups; g++) {
+      float v = -INFINITY;
+#pragma unroll
+      for (int sI = 0; sI < MOE_MAX_SLOTS; sI++) {
+        const int e = lane + 32 * sI;
+        if (e < E && e / gsz == g) v = fmaxf(v, sc[sI]);
+      }
+      v = warp_max(v);
+#pragma unroll
+      for (int sI = 0; sI < MOE_MAX_SLOTS; sI++)
+        if (lane + 32 * sI == g) gb[sI] = v;
+    }
+    for (int k = 0; k < p.groups_keep; k++) {
+      float best = -INFINITY;
+      int bi = 0x7fffffff;
+#pragma unroll
+      for (int sI = 0; sI < MOE_MAX_SLOTS; sI++)
+        if (gb[sI] > best) { best = gb[sI]; bi = lane + 32 * sI; }
+#pragma unroll
+      for (int o = 16; o > 0; o >>= 1) {
+        const float ob = __shfl_xor_sync(0xffffffffu, best, o);
+        const int oi = __shfl_xor_sync(0xffffffffu, bi, o);
+        if (ob > best || (ob == best && oi < bi)) { best = ob; bi = oi; }
+      }
+#pragma unroll
+      for (int sI = 0; sI < MOE_MAX_SLOTS; sI++) {
+        if (lane + 32 * sI == bi) gb[sI] = -INFINITY;
+        if ((lane + 32 * sI) / gsz == bi) open[sI] = true;
+      }
+    }
+#pragma unroll
+    for (int sI = 0; sI < MOE_MAX_SLOTS; sI++)
+      if (!open[sI]) ch[sI] = -INFINITY;
   }
   float wsum = 0.f, mine = 0.f;  // lane k keeps the score of the k-th choice
   int mine_id = 0;
@@ -947,7 +987,7 @@ __global__ void __launch_bounds__(128) moe_router_kernel(const MoePlan p) {
   }
   if (lane < p.top) {
     p.ids[(size_t)m * p.top + lane] = mine_id;
-    p.wts[(size_t)m * p.top + lane] = mine / (wsum + 1e-20f) * p.scale;
+    p.wts[(size_t)m * p.top + lane] = (p.plain_weights ? mine : mine / (wsum + 1e-20f)) * p.scale;
   }
   if (p.has_shared_gate && lane == 0) p.sgate[m] = 1.0f / (1.0f + expf(-lg[E]));
 }
@@ -1023,6 +1063,10 @@ __global__ void __launch_bounds__(256) moe_plan_small_kernel(const MoePlan p) {
 }
 int moe_route(cudaStream_t st, int dtype, const MoePlan &p, uint64_t *launches) {
   if (p.experts + p.identity > 32 * MOE_MAX_SLOTS || p.top > 32 || p.top < 1 || p.top > p.experts + p.identity) return (int)cudaErrorInvalidValue;
+  if (p.groups > 1 && (p.identity > 0 || p.logit_bias || p.experts % p.groups || p.groups_keep < 1 || p.groups_keep > p.groups ||
+                       p.top > p.groups_keep * (p.experts / p.groups)))
+    return (int)cudaErrorInvalidValue;
+  if (p.logit_bias && !p.correction) return (int)cudaErrorInvalidValue;
   MX_DISPATCH(dtype, (moe_router_kernel<T><<<(p.M + 3) / 4, 128, 0, st>>>(p)));
   int n = 1;
   if (p.experts > 0 && p.M * p.top <= MOE_SMALL_PAIRS) {
@@ -1129,8 +1173,8 @@ __global__ void __launch_bounds__(256) moe_expert_kernel(const MoeExperts p) {
       const int n = n0 + tx * 4 + j;
       if (n >= N) continue;
       if (PHASE == 0) {
-        if (p.act_kind == 2) {
-          reinterpret_cast<T *>(p.act)[(size_t)(row0 + r) * p.ff + n] = DT<T>::from_f(gated_pair<T>(acc[i][j], acu[i][j], 2, p.limit));
+        if (p.act_kind >= 2) {
+          reinterpret_cast<T *>(p.act)[(size_t)(row0 + r) * p.ff + n] = DT<T>::from_f(gated_pair<T>(acc[i][j], acu[i][j], p.act_kind, p.limit));
           continue;
         }
         const float g = rnd<T>(act_f(rnd<T>(acc[i][j]), p.act_kind));
@@ -1364,6 +1408,107 @@ int branch_merge(cudaStream_t st, int dtype, const BranchMerge &p, uint64_t *lau
       if (e != cudaSuccess) return (int)e;
     }
     branch_merge_kernel<T><<<p.M, 256, smem, st>>>(p);
+  });
+  MX_DONE(1);
+}
+
+// ---------------------------------------------------------------------------------------------- sublayer output -> stream, one pass
+// A CTA per row; the row of y stays in registers between its sum of squares and its way into the stream: thread i owns the
+// 16-byte pieces i, i + 256, ... (NV of them).  Widths beyond the register form, or no multiples of four, keep y in shared memory.
+template <typename T> __device__ __forceinline__ float4 merge_load(const StreamMerge &p, int m, int i4) {
+  if (p.a) return reinterpret_cast<const float4 *>(p.a + (size_t)m * p.n)[i4];
+  float4 s = make_float4(0.f, 0.f, 0.f, 0.f);
+  for (int k = 0; k < p.top; k++) {
+    const size_t pr = (size_t)m * p.top + k;
+    if (p.ids[pr] >= p.experts) continue;
+    const float w = p.wts[pr];
+    const float4 y = reinterpret_cast<const float4 *>(p.y + (size_t)p.pos_of[pr] * p.n)[i4];
+    s.x = fmaf(w, y.x, s.x); s.y = fmaf(w, y.y, s.y); s.z = fmaf(w, y.z, s.z); s.w = fmaf(w, y.w, s.w);
+  }
+  return s;
+}
+template <typename T, int NV>
+__global__ void __launch_bounds__(256) stream_merge_kernel(const StreamMerge p) {
+  __shared__ float red[64];
+  const int m = blockIdx.x, n4 = p.n / 4;
+  const T *post = reinterpret_cast<const T *>(p.post);
+  const float4 *x4 = reinterpret_cast<const float4 *>(p.x + (size_t)m * p.n);
+  float4 y[NV], xv[NV];
+  float ss = 0.f, z = 0.f;
+#pragma unroll
+  for (int v = 0; v < NV; v++) {
+    const int i = threadIdx.x + 256 * v;
+    y[v] = xv[v] = make_float4(0.f, 0.f, 0.f, 0.f);
+    if (i < n4) {
+      y[v] = merge_load<T>(p, m, i);
+      xv[v] = x4[i];
+    }
+    ss = fmaf(y[v].x, y[v].x, ss); ss = fmaf(y[v].y, y[v].y, ss); ss = fmaf(y[v].z, y[v].z, ss); ss = fmaf(y[v].w, y[v].w, ss);
+  }
+  float inv = 1.f;
+  if (post) {
+    block_sum2(ss, z, red);
+    inv = 1.0f / sqrtf(ss / (float)p.n + p.eps);
+  }
+#pragma unroll
+  for (int v = 0; v < NV; v++) {
+    const int i = threadIdx.x + 256 * v;
+    if (i >= n4) continue;
+    float r[4] = {y[v].x, y[v].y, y[v].z, y[v].w};
+    if (post) {
+#pragma unroll
+      for (int e = 0; e < 4; e++) r[e] = r[e] * inv * DT<T>::to_f(post[4 * i + e]);
+    }
+    r[0] += xv[v].x; r[1] += xv[v].y; r[2] += xv[v].z; r[3] += xv[v].w;
+    reinterpret_cast<float4 *>(p.x_out + (size_t)m * p.n)[i] = make_float4(r[0], r[1], r[2], r[3]);
+    if (p.xd) store4<T>(reinterpret_cast<T *>(p.xd) + (size_t)m * p.n + 4 * i, r);
+  }
+}
+template <typename T>
+__global__ void __launch_bounds__(256) stream_merge_any_kernel(const StreamMerge p) {
+  extern __shared__ float ys[];  // [n]
+  __shared__ float red[64];
+  const int m = blockIdx.x;
+  const T *post = reinterpret_cast<const T *>(p.post);
+  float ss = 0.f, z = 0.f;
+  for (int i = threadIdx.x; i < p.n; i += blockDim.x) {
+    float v = 0.f;
+    if (p.a) v = p.a[(size_t)m * p.n + i];
+    else
+      for (int k = 0; k < p.top; k++) {
+        const size_t pr = (size_t)m * p.top + k;
+        if (p.ids[pr] < p.experts) v = fmaf(p.wts[pr], p.y[(size_t)p.pos_of[pr] * p.n + i], v);
+      }
+    ys[i] = v;
+    ss = fmaf(v, v, ss);
+  }
+  float inv = 1.f;
+  if (post) {
+    block_sum2(ss, z, red);
+    inv = 1.0f / sqrtf(ss / (float)p.n + p.eps);
+  }
+  for (int i = threadIdx.x; i < p.n; i += blockDim.x) {  // a thread revisits the entries it wrote
+    const float r = p.x[(size_t)m * p.n + i] + (post ? ys[i] * inv * DT<T>::to_f(post[i]) : ys[i]);
+    p.x_out[(size_t)m * p.n + i] = r;
+    if (p.xd) reinterpret_cast<T *>(p.xd)[(size_t)m * p.n + i] = DT<T>::from_f(r);
+  }
+}
+int stream_merge(cudaStream_t st, int dtype, const StreamMerge &p, uint64_t *launches) {
+  if (p.M < 1 || p.n < 1 || !p.x || !p.x_out || (!p.a && (!p.y || !p.wts || !p.ids || !p.pos_of || p.top < 1))) return (int)cudaErrorInvalidValue;
+  const bool vec = p.n % 4 == 0 && p.n <= 8192 && (((uintptr_t)p.a | (uintptr_t)p.y | (uintptr_t)p.x | (uintptr_t)p.x_out | (uintptr_t)p.xd) & 15) == 0;
+  const size_t smem = (size_t)p.n * sizeof(float);
+  if (!vec && smem > 200 * 1024) return (int)cudaErrorInvalidValue;
+  MX_DISPATCH(dtype, {
+    if (!vec) {
+      if (smem > 48 * 1024) {
+        cudaError_t e = cudaFuncSetAttribute(stream_merge_any_kernel<T>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+        if (e != cudaSuccess) return (int)e;
+      }
+      stream_merge_any_kernel<T><<<p.M, 256, smem, st>>>(p);
+    } else if (p.n <= 1024) stream_merge_kernel<T, 1><<<p.M, 256, 0, st>>>(p);
+    else if (p.n <= 2048) stream_merge_kernel<T, 2><<<p.M, 256, 0, st>>>(p);
+    else if (p.n <= 4096) stream_merge_kernel<T, 4><<<p.M, 256, 0, st>>>(p);
+    else stream_merge_kernel<T, 8><<<p.M, 256, 0, st>>>(p);
   });
   MX_DONE(1);
 }
@@ -2185,6 +2330,28 @@ __global__ void __launch_bounds__(128) embed_tables_kernel(const EmbedTables p) 
 int embed_tables(cudaStream_t st, int dtype, const EmbedTables &p, uint64_t *launches) {
   if (p.B < 1 || p.S < 1 || (p.bigram && p.buckets < 1)) return (int)cudaErrorInvalidValue;
   MX_DISPATCH(dtype, (embed_tables_kernel<T><<<p.B * p.S, 128, 0, st>>>(p)));
+  MX_DONE(1);
+}
+// token row, RMS norm over the width with a gain
+template <typename T>
+__global__ void __launch_bounds__(256) embed_norm_kernel(const T *__restrict__ E, const uint32_t *__restrict__ ids, const T *__restrict__ w,
+                                                         float *__restrict__ x, int W, float scale, float eps) {
+  __shared__ float red[64];
+  const T *row = E + (size_t)ids[blockIdx.x] * W;
+  float *out = x + (size_t)blockIdx.x * W;
+  float ss = 0.f, z = 0.f;
+  for (int i = threadIdx.x; i < W; i += blockDim.x) {
+    const float v = DT<T>::to_f(row[i]) * scale;
+    ss = fmaf(v, v, ss);
+  }
+  block_sum2(ss, z, red);
+  const float inv = 1.0f / sqrtf(ss / (float)W + eps);
+  for (int i = threadIdx.x; i < W; i += blockDim.x) out[i] = DT<T>::to_f(row[i]) * scale * inv * DT<T>::to_f(w[i]);
+}
+int embed_norm(cudaStream_t st, int dtype, const void *E, const uint32_t *ids, const void *w, float *x, int M, int W, int vocab, float scale, float eps,
+               uint64_t *launches) {
+  if (M < 1 || W < 1 || vocab < 1 || !E || !ids || !w || !x) return (int)cudaErrorInvalidValue;
+  MX_DISPATCH(dtype, (embed_norm_kernel<T><<<M, 256, 0, st>>>(reinterpret_cast<const T *>(E), ids, reinterpret_cast<const T *>(w), x, W, scale != 0.f ? scale : 1.f, eps)));
   MX_DONE(1);
 }
 

@@ -124,6 +124,8 @@ struct GateNorm {
   int gate_sigmoid = 0;            // 1: the gate is sigmoid(gate) instead of silu(gate)
   int w_period = 0;                // > 0: w has w_period entries and repeats (one gain vector shared by every part)
   const float *row_div = nullptr;  // [M, parts] fp32: o of a part is divided by its entry before anything else
+  int ldo = 0;                     // row stride of out when it is a column range of a wider buffer (0 = n)
+  float out_scale = 1.f;           // a constant factor of the output
 };
 int gate_norm(cudaStream_t, int dtype, const GateNorm &, uint64_t *launches);
 
@@ -150,6 +152,9 @@ struct MoePlan {
   // 1: `correction` is a bias of the logits (z = Wr h + correction); the `top` largest z are chosen and their weights are the
   // softmax over the chosen z alone (times scale)
   int logit_bias = 0;
+  // groups > 1: the experts form that many equal groups of neighbours, only those of the groups_keep groups with the largest best
+  // score s may be chosen; plain_weights: the weights are the scores s (times scale), not renormalised.  correction may be nullptr
+  int groups = 0, groups_keep = 0, plain_weights = 0;
 };
 int moe_route(cudaStream_t, int dtype, const MoePlan &, uint64_t *launches);
 
@@ -218,6 +223,23 @@ struct BranchMerge {
   float eps;
 };
 int branch_merge(cudaStream_t, int dtype, const BranchMerge &, uint64_t *launches);
+
+// The same way back into the stream for a sublayer without branch norms, in one pass over the row:
+//   y = a   or, with MoE outputs, y = sum over slots of wts * y_sorted[pos_of]  (slots in order; no identity experts)
+//   x_out = x + (post ? rms(y) * post : y);   xd (nullable) = x_out rounded to D: the next sublayer's operand
+struct StreamMerge {
+  const float *a;        // [M, n] fp32, or nullptr with the routed sum below
+  const float *y, *wts;  // [sorted rows, n], [M, top]
+  const int *ids, *pos_of;  // [M, top]; slots whose id is not below `experts` add nothing
+  int top, experts;
+  const void *post;      // [n] D or nullptr
+  const float *x;
+  float *x_out;          // may alias x
+  void *xd;              // [M, n] D or nullptr
+  int M, n;
+  float eps;
+};
+int stream_merge(cudaStream_t, int dtype, const StreamMerge &, uint64_t *launches);
 
 // ---- gated delta rule -----------------------------------------------------------------------------------------------------
 // Prep: q and k of every key head become unit vectors (x / sqrt(sum x^2 + 1e-6); q also times qscale) in fp32, and per head
@@ -326,6 +348,9 @@ struct EmbedTables {
   float scale;           // 0 = none
 };
 int embed_tables(cudaStream_t, int dtype, const EmbedTables &, uint64_t *launches);
+// x[m] = rms(E[ids[m]] * scale) * w      (scale 0 = none; fp32 stream)
+int embed_norm(cudaStream_t, int dtype, const void *E, const uint32_t *ids, const void *w, float *x, int M, int W, int vocab, float scale, float eps,
+               uint64_t *launches);
 
 // ---- x[m] += (x0 ? x0[m] : 0) + vec   (fp32 stream; vec [W] in D) --------------------------------------------------------
 int stream_inject(cudaStream_t, int dtype, float *x, const float *x0, const void *vec, int M, int W, uint64_t *launches);
@@ -372,10 +397,23 @@ struct QkPrep {
   void *q_out;           // [M, heads * dim] D
   void *kc, *vc;         // [B, kv_heads, cap, dim], [B, kv_heads, cap, vdim] D
   int B, S, heads, kv_heads, dim, vdim, cap, pos0;
+  int interleaved = 0;   // 1: pairs (2i, 2i + 1) instead of (i, i + rope_dims / 2)
+  const void *q_w = nullptr, *k_w = nullptr;  // [dim] D: every head is x / rms(x) * gain IN FRONT OF the rotation (instead of unit_norm)
+  int v_unit = 0;        // 1: every value head is divided by its root mean square
 };
 int qk_prep(cudaStream_t, int dtype, const QkPrep &, uint64_t *launches);
 
+// ---- means over complete blocks of cached rows ----------------------------------------------------------------------------------
+// Blocks of `pool` positions that positions [pos0, pos0 + S) complete: pk[b, g, blk] = mean of the block's rows of kc, pv likewise.
+struct PoolRows {
+  const void *kc, *vc;   // [B, kv_heads, cap, dim], [B, kv_heads, cap, vdim] D
+  void *pk, *pv;         // [B, kv_heads, pcap, dim], [B, kv_heads, pcap, vdim] D
+  int B, S, kv_heads, dim, vdim, cap, pcap, pos0, pool;
+};
+int pool_rows(cudaStream_t, int dtype, const PoolRows &, uint64_t *launches);  // launches nothing when no block completes
+
 // ---- softmax attention over cached keys and values with a sliding window, kept first tokens and a sink -----------------------
+// (optionally pooled blocks in front of the window, or chunks of fixed places)
 // Row i (absolute position) of head h sees key j of key head h / (heads / kv_heads) when j <= i and (window == 0 or i - j < window
 // or j < keep_first).  s = (q . k_j) * scale; w_j = exp(s_j) / (sum over visible exp(s) + (sink ? exp(sink[h]) : 0)); the sink has
 // no value.  out_h = (sum_j w_j v_j) * sigmoid(gate) with one gate per entry (gate_per_head 0: column h * vdim + e) or per head
@@ -395,6 +433,12 @@ struct WindowAttn {
   // weighted values) land in part [M * heads, nsplit, vdim + 2] fp32 and are merged by a second kernel
   float *part = nullptr;
   int nsplit = 0;
+  // pool > 0 (with a window): block blk of `pool` positions is one more key (row blk of pk / pv, [B, kv_heads, pcap, dim | vdim]) once
+  // (blk + 1) pool <= i - window + 1.  chunk > 0: j >= i / chunk * chunk.  softcap > 0: s <- softcap tanh(s / softcap).  sink_zero: the
+  // denominator holds exp(0).  out_scale: a constant factor of the output
+  const void *pk = nullptr, *pv = nullptr;
+  int pool = 0, pcap = 0, chunk = 0, sink_zero = 0;
+  float softcap = 0.f, out_scale = 1.f;
 };
 int window_attention(cudaStream_t, int dtype, const WindowAttn &, uint64_t *launches);
 // The tiled form for portions in 16-bit D (tensor-core products, a CTA per 64 rows of a head): true when the shapes fit it.

@@ -1,6 +1,6 @@
 // mixers_window.cu — kernels behind the second half of mixers.cuh: the element-wise squashing norm, RMS norms of column ranges
-// (low-rank latents), rotation + unit norm of queries and keys with the cache append, softmax attention over cached keys and
-// values with a sliding window, kept first tokens and a sink (per-row form with split keys for short steps, and a tiled
+// (low-rank latents), rotation + norms of queries, keys and values with the cache append, means of blocks of cached rows, softmax
+// attention over cached keys and values with a sliding window or chunks, pooled blocks, kept first tokens and a sink (per-row form with split keys for short steps, and a tiled
 // tensor-core form for portions in 16-bit D), the per-layer token input and the stream / embedding concatenation.
 // sm_100a only.  fp32 everywhere the interface says so; D only where a projection, a cache row or a weight is stored.
 #include "mixers.cuh"
@@ -28,6 +28,8 @@ namespace mx {
     return (int)cudaGetLastError();    \
   } while (0)
 
+template <typename T> struct Bits16 { typedef T type; };
+template <> struct Bits16<float> { typedef __nv_bfloat16 type; };  // never taken for float (sizeof test); keeps the vector path instantiable
 __device__ __forceinline__ float sigmoid_f(float z) { return 1.0f / (1.0f + expf(-z)); }
 
 // ---------------------------------------------------------------------------------------------- squashing norm
@@ -97,10 +99,19 @@ int rms_cols(cudaStream_t st, int dtype, const RmsCols &p, uint64_t *launches) {
 }
 
 // ---------------------------------------------------------------------------------------------- rotation, unit norm, append
-// entry i of a head whose first `dims` entries are paired (i, i + dims / 2); cs / sn: this position's table row
+// entry i of a head whose first `dims` entries are paired (i, i + dims / 2), or (2i, 2i + 1) when interleaved; cs / sn: this
+// position's table row; w: gains multiplied onto the entries before they turn, or nullptr
 template <typename T>
-__device__ __forceinline__ float rotated_entry(const T *v, int i, int dims, const float *cs, const float *sn) {
+__device__ __forceinline__ float rotated_entry(const T *v, int i, int dims, const float *cs, const float *sn, const T *w, bool inter) {
   const int half = dims >> 1;
+  if (w || inter) {
+    const float x = DT<T>::to_f(v[i]) * (w ? DT<T>::to_f(w[i]) : 1.f);
+    if (i >= dims) return x;
+    const bool first = inter ? (i & 1) == 0 : i < half;
+    const int j = inter ? i ^ 1 : (first ? i + half : i - half), f = inter ? i >> 1 : (first ? i : j);
+    const float y = DT<T>::to_f(v[j]) * (w ? DT<T>::to_f(w[j]) : 1.f);
+    return first ? x * cs[f] - y * sn[f] : x * cs[f] + y * sn[f];
+  }
   if (i >= dims) return DT<T>::to_f(v[i]);
   if (i < half) return DT<T>::to_f(v[i]) * cs[i] - DT<T>::to_f(v[i + half]) * sn[i];
   return DT<T>::to_f(v[i]) * cs[i - half] + DT<T>::to_f(v[i - half]) * sn[i - half];
@@ -119,16 +130,28 @@ __global__ void __launch_bounds__(256) qk_prep_kernel(const QkPrep p) {
     T *o = is_q ? reinterpret_cast<T *>(p.q_out) + ((size_t)m * p.heads + hv) * p.dim
                 : reinterpret_cast<T *>(p.kc) + (((size_t)b * p.kv_heads + g) * p.cap + pos) * p.dim;
     float inv = 1.f;
-    if (p.unit_norm) {
+    const T *w = reinterpret_cast<const T *>(is_q ? p.q_w : p.k_w);
+    if (p.unit_norm || w) {
       float ss = 0.f;
-      for (int i = lane; i < p.dim; i += 32) {
-        const float r = rotated_entry<T>(v, i, dims, cs, sn);
+      for (int i = lane; i < p.dim; i += 32) {  // a rotation keeps the length: with gains, the norm is that of the entries as they come
+        const float r = w ? DT<T>::to_f(v[i]) : rotated_entry<T>(v, i, dims, cs, sn, w, p.interleaved != 0);
         ss = fmaf(r, r, ss);
       }
       ss = warp_sum(ss);
       inv = 1.0f / sqrtf(ss / (float)p.dim + p.eps);
     }
-    for (int i = lane; i < p.dim; i += 32) o[i] = DT<T>::from_f(rotated_entry<T>(v, i, dims, cs, sn) * inv);
+    for (int i = lane; i < p.dim; i += 32) o[i] = DT<T>::from_f(rotated_entry<T>(v, i, dims, cs, sn, w, p.interleaved != 0) * inv);
+  }
+  if (p.v_unit) {
+    for (int g = warp; g < p.kv_heads; g += nw) {
+      const T *v = row + p.v_col + (size_t)g * p.vdim;
+      T *o = reinterpret_cast<T *>(p.vc) + (((size_t)b * p.kv_heads + g) * p.cap + pos) * p.vdim;
+      float ss = 0.f;
+      for (int i = lane; i < p.vdim; i += 32) ss = fmaf(DT<T>::to_f(v[i]), DT<T>::to_f(v[i]), ss);
+      const float inv = 1.0f / sqrtf(warp_sum(ss) / (float)p.vdim + p.eps);
+      for (int i = lane; i < p.vdim; i += 32) o[i] = DT<T>::from_f(DT<T>::to_f(v[i]) * inv);
+    }
+    return;
   }
   for (int i = threadIdx.x; i < p.kv_heads * p.vdim; i += blockDim.x) {
     const int g = i / p.vdim, e = i % p.vdim;
@@ -175,22 +198,53 @@ __global__ void __launch_bounds__(256) qk_prep_vec_kernel(const QkPrep p) {
       r[2 * q] = f.x;
       r[2 * q + 1] = f.y;
     }
-    if (i0 < dims) {
+    const T *wn = reinterpret_cast<const T *>(is_q ? p.q_w : p.k_w);
+    float inv = 1.f;
+    if (wn) {  // RMS norm with gains in front of the rotation
+      float ss = 0.f;
+#pragma unroll
+      for (int q = 0; q < E; q++) ss = fmaf(r[q], r[q], ss);
+      inv = 1.0f / sqrtf(warp_sum(ss) / (float)p.dim + p.eps);
+      uint32_t ww[E / 2];
+      load_words<E>(wn + i0, ww);
+#pragma unroll
+      for (int q = 0; q < E / 2; q++) {
+        const float2 f = DT<T>::unpack2(ww[q]);
+        r[2 * q] *= f.x;
+        r[2 * q + 1] *= f.y;
+      }
+    }
+    if (p.interleaved) {
+      if (i0 < dims) {
+#pragma unroll
+        for (int q = 0; q < E / 2; q++) {
+          const float c = cs[(i0 >> 1) + q], sfac = sn[(i0 >> 1) + q], u = r[2 * q];
+          r[2 * q] = u * c - r[2 * q + 1] * sfac;
+          r[2 * q + 1] = r[2 * q + 1] * c + u * sfac;
+        }
+      }
+    } else if (i0 < dims) {
       const bool lo = i0 < half;
       uint32_t wb[E / 2];
       load_words<E>(v + (lo ? i0 + half : i0 - half), wb);
       float c[E], sfac[E];
       load_floats<E>(cs + (lo ? i0 : i0 - half), c);
       load_floats<E>(sn + (lo ? i0 : i0 - half), sfac);
+      uint32_t wg[E / 2];
+      if (wn) load_words<E>(wn + (lo ? i0 + half : i0 - half), wg);
 #pragma unroll
       for (int q = 0; q < E / 2; q++) {
-        const float2 f = DT<T>::unpack2(wb[q]);
+        float2 f = DT<T>::unpack2(wb[q]);
+        if (wn) {
+          const float2 g2 = DT<T>::unpack2(wg[q]);
+          f.x *= g2.x;
+          f.y *= g2.y;
+        }
         r[2 * q] = lo ? r[2 * q] * c[2 * q] - f.x * sfac[2 * q] : r[2 * q] * c[2 * q] + f.x * sfac[2 * q];
         r[2 * q + 1] = lo ? r[2 * q + 1] * c[2 * q + 1] - f.y * sfac[2 * q + 1] : r[2 * q + 1] * c[2 * q + 1] + f.y * sfac[2 * q + 1];
       }
     }
-    float inv = 1.f;
-    if (p.unit_norm) {
+    if (p.unit_norm && !wn) {
       float ss = 0.f;
 #pragma unroll
       for (int q = 0; q < E; q++) ss = fmaf(r[q], r[q], ss);
@@ -204,6 +258,27 @@ __global__ void __launch_bounds__(256) qk_prep_vec_kernel(const QkPrep p) {
     else if (E == 4) *reinterpret_cast<uint2 *>(o + i0) = make_uint2(wo[0], wo[1]);
     else *reinterpret_cast<uint4 *>(o + i0) = make_uint4(wo[0], wo[E / 2 > 1 ? 1 : 0], wo[E / 2 > 2 ? 2 : 0], wo[E / 2 > 3 ? 3 : 0]);
   }
+  if (p.v_unit) {  // a warp per value head, 16-byte pieces (two passes; the second comes out of L1)
+    for (int g = warp; g < p.kv_heads; g += nw) {
+      const T *v = row + p.v_col + (size_t)g * p.vdim;
+      T *o = reinterpret_cast<T *>(p.vc) + (((size_t)b * p.kv_heads + g) * p.cap + pos) * p.vdim;
+      float ss = 0.f;
+      for (int i = lane * 8; i < p.vdim; i += 256) {
+        float f[8];
+        unpack8<T>(*reinterpret_cast<const uint4 *>(v + i), f);
+#pragma unroll
+        for (int e = 0; e < 8; e++) ss = fmaf(f[e], f[e], ss);
+      }
+      const float inv = 1.0f / sqrtf(warp_sum(ss) / (float)p.vdim + p.eps);
+      for (int i = lane * 8; i < p.vdim; i += 256) {
+        float f[8];
+        unpack8<T>(*reinterpret_cast<const uint4 *>(v + i), f);
+        *reinterpret_cast<uint4 *>(o + i) = make_uint4(pack2x<T>(f[0] * inv, f[1] * inv), pack2x<T>(f[2] * inv, f[3] * inv),
+                                                       pack2x<T>(f[4] * inv, f[5] * inv), pack2x<T>(f[6] * inv, f[7] * inv));
+      }
+    }
+    return;
+  }
   const int vrow = p.kv_heads * p.vdim;  // values: 16-byte pieces (vdim, v_col multiples of 8)
   for (int i = threadIdx.x * 8; i < vrow; i += blockDim.x * 8) {
     const int g = i / p.vdim, e = i % p.vdim;
@@ -213,10 +288,11 @@ __global__ void __launch_bounds__(256) qk_prep_vec_kernel(const QkPrep p) {
 }
 template <typename T> static bool qk_prep_vec(cudaStream_t st, const QkPrep &p) {
   const int E = p.dim / 32, half = p.cos_t ? p.rope_dims / 2 : 0;
-  const bool ok = p.dim % 32 == 0 && (E == 2 || E == 4 || E == 8) && half % E == 0 && p.vdim % 8 == 0 && p.ld % 8 == 0 && p.q_col % 8 == 0 &&
+  const bool ok = p.dim % 32 == 0 && (E == 2 || E == 4 || E == 8) && (p.interleaved ? 2 * half : half) % E == 0 && p.vdim % 8 == 0 && p.ld % 8 == 0 && p.q_col % 8 == 0 &&
                   p.k_col % 8 == 0 && p.v_col % 8 == 0 &&
-                  (((uintptr_t)p.proj | (uintptr_t)p.q_out | (uintptr_t)p.kc | (uintptr_t)p.vc | (uintptr_t)p.cos_t | (uintptr_t)p.sin_t) & 15) == 0 &&
-                  (half * sizeof(float)) % 16 == 0;
+                  (((uintptr_t)p.proj | (uintptr_t)p.q_out | (uintptr_t)p.kc | (uintptr_t)p.vc | (uintptr_t)p.cos_t | (uintptr_t)p.sin_t | (uintptr_t)p.q_w |
+                    (uintptr_t)p.k_w) & 15) == 0 &&
+                  (p.interleaved || (half * sizeof(float)) % 16 == 0);
   if (!ok) return false;
   const unsigned nt = (p.heads + p.kv_heads) > 4 ? 256 : 128;
   if (E == 2) qk_prep_vec_kernel<T, 2><<<p.B * p.S, nt, 0, st>>>(p);
@@ -226,7 +302,7 @@ template <typename T> static bool qk_prep_vec(cudaStream_t st, const QkPrep &p) 
 }
 template <> bool qk_prep_vec<float>(cudaStream_t, const QkPrep &) { return false; }
 int qk_prep(cudaStream_t st, int dtype, const QkPrep &p, uint64_t *launches) {
-  if (p.B < 1 || p.S < 1 || p.heads < 1 || p.kv_heads < 1 || (p.cos_t && (p.rope_dims & 1 || p.rope_dims > p.dim))) return (int)cudaErrorInvalidValue;
+  if (p.B < 1 || p.S < 1 || p.heads < 1 || p.kv_heads < 1 || !p.q_w != !p.k_w || (p.cos_t && (p.rope_dims & 1 || p.rope_dims > p.dim))) return (int)cudaErrorInvalidValue;
   bool done = false;
   MX_DISPATCH(dtype, (done = qk_prep_vec<T>(st, p)));
   if (done) MX_DONE(1);
@@ -234,8 +310,60 @@ int qk_prep(cudaStream_t st, int dtype, const QkPrep &p, uint64_t *launches) {
   MX_DONE(1);
 }
 
+// ---------------------------------------------------------------------------------------------- means of blocks of cached rows
+// CTA (block, key head, batch row): threads own columns of the key row, then of the value row; E adjacent ones at a time
+template <typename T, int E>
+__global__ void __launch_bounds__(128) pool_rows_kernel(const PoolRows p) {
+  const int blk = p.pos0 / p.pool + blockIdx.x, g = blockIdx.y, b = blockIdx.z;
+  const size_t bg = (size_t)b * p.kv_heads + g;
+  const float inv = 1.0f / (float)p.pool;
+  for (int i = threadIdx.x * E; i < p.dim + p.vdim; i += blockDim.x * E) {
+    const bool key = i < p.dim;
+    const int c = key ? i : i - p.dim, w = key ? p.dim : p.vdim;
+    const T *src = reinterpret_cast<const T *>(key ? p.kc : p.vc) + (bg * p.cap + (size_t)blk * p.pool) * w + c;
+    T *dst = reinterpret_cast<T *>(key ? p.pk : p.pv) + (bg * p.pcap + blk) * w + c;
+    float s[E];
+#pragma unroll
+    for (int e = 0; e < E; e++) s[e] = 0.f;
+    for (int r = 0; r < p.pool; r++) {
+      if (E == 4 && sizeof(T) == 2) {
+        const uint2 u = *reinterpret_cast<const uint2 *>(src + (size_t)r * w);
+        typedef typename Bits16<T>::type B;
+        const float2 a = DT<B>::unpack2(u.x), d = DT<B>::unpack2(u.y);
+        s[0] += a.x; s[E > 1 ? 1 : 0] += a.y; s[E > 2 ? 2 : 0] += d.x; s[E > 3 ? 3 : 0] += d.y;
+      } else {
+#pragma unroll
+        for (int e = 0; e < E; e++) s[e] += DT<T>::to_f(src[(size_t)r * w + e]);
+      }
+    }
+#pragma unroll
+    for (int e = 0; e < E; e++) dst[e] = DT<T>::from_f(s[e] * inv);
+  }
+}
+int pool_rows(cudaStream_t st, int dtype, const PoolRows &p, uint64_t *launches) {
+  if (p.pool < 1 || p.B < 1 || p.S < 1 || !p.kc || !p.vc || !p.pk || !p.pv || p.pos0 + p.S > p.cap || (p.pos0 + p.S) / p.pool > p.pcap)
+    return (int)cudaErrorInvalidValue;
+  const int n = (p.pos0 + p.S) / p.pool - p.pos0 / p.pool;
+  if (n < 1) return 0;
+  const bool vec = p.dim % 4 == 0 && p.vdim % 4 == 0 && (((uintptr_t)p.kc | (uintptr_t)p.vc | (uintptr_t)p.pk | (uintptr_t)p.pv) & 15) == 0;
+  MX_DISPATCH(dtype, {
+    if (vec) pool_rows_kernel<T, 4><<<dim3(n, p.kv_heads, p.B), 128, 0, st>>>(p);
+    else pool_rows_kernel<T, 1><<<dim3(n, p.kv_heads, p.B), 128, 0, st>>>(p);
+  });
+  MX_DONE(1);
+}
+
 // ---------------------------------------------------------------------------------------------- window attention, per row
-// CTA (row-head, split): the visible keys are the kept first tokens that have left the window, then the window; the CTA's
+// blocks of pooled positions that row `pos` sees: those that end at least `window` positions back
+__device__ __forceinline__ int pooled_seen(int pos, int window, int pool) {
+  return pool > 0 && window > 0 && pos >= window ? (pos - window + 1) / pool : 0;
+}
+// the first position that row `pos` sees through its window and its chunk
+__device__ __forceinline__ int first_seen(int pos, int window, int chunk) {
+  const int lo = window > 0 ? max(0, pos - window + 1) : 0;
+  return chunk > 0 ? max(lo, pos / chunk * chunk) : lo;
+}
+// CTA (row-head, split): the visible keys are the pooled blocks, the kept first tokens that have left the window, then the window; the CTA's
 // four warps walk its share four keys at a time each (lanes split the columns of a key and of a value row), their running
 // softmax states are merged in shared memory.  Without splits the CTA adds the sink, normalises, gates and writes the output;
 // with splits it leaves (max, sum, weighted values) for the merge kernel.
@@ -246,15 +374,17 @@ __global__ void __launch_bounds__(128) window_attn_kernel(const WindowAttn p) {
   const int mh = blockIdx.x, split = blockIdx.y, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int m = mh / p.heads, h = mh % p.heads, b = m / p.S, t = m % p.S, pos = p.pos0 + t;
   const int g = h / (p.heads / p.kv_heads);
-  const int lo = p.window > 0 ? max(0, pos - p.window + 1) : 0;
-  const int nA = min(p.keep_first, lo), total = nA + pos - lo + 1;
+  const int lo = first_seen(pos, p.window, p.chunk);
+  const int nP = pooled_seen(pos, p.window, p.pool), nA = nP + min(p.keep_first, lo), total = nA + pos - lo + 1;
   const int nsplit = p.nsplit > 1 ? p.nsplit : 1;
   const int per = nsplit > 1 ? ((total + nsplit - 1) / nsplit + 15) / 16 * 16 : total;
   const int k0 = split * per, k1 = min(total, k0 + per);
   const T *q = reinterpret_cast<const T *>(p.q) + (size_t)m * p.ldq + (size_t)h * p.dim;
   const T *kc = reinterpret_cast<const T *>(p.kc) + ((size_t)b * p.kv_heads + g) * p.cap * p.dim;
   const T *vc = reinterpret_cast<const T *>(p.vc) + ((size_t)b * p.kv_heads + g) * p.cap * p.vdim;
-  const bool shared_rows = p.kc == p.vc && p.dim == p.vdim;  // a key row is also the value row
+  const T *pk = p.pool > 0 ? reinterpret_cast<const T *>(p.pk) + ((size_t)b * p.kv_heads + g) * p.pcap * p.dim : nullptr;
+  const T *pv = p.pool > 0 ? reinterpret_cast<const T *>(p.pv) + ((size_t)b * p.kv_heads + g) * p.pcap * p.vdim : nullptr;
+  const bool shared_rows = p.kc == p.vc && p.dim == p.vdim && p.pool == 0;  // a key row is also the value row
   float qv[NR], acc[NR];
 #pragma unroll
   for (int i = 0; i < NR; i++) {
@@ -268,8 +398,9 @@ __global__ void __launch_bounds__(128) window_attn_kernel(const WindowAttn p) {
 #pragma unroll
     for (int u = 0; u < 4; u++) {
       const int ju = jj + u < k1 ? jj + u : jj;
-      const int j = ju < nA ? ju : lo + ju - nA;
-      const T *krow = kc + (size_t)j * p.dim;
+      const bool pooled = ju < nP;
+      const int j = ju < nA ? (pooled ? ju : ju - nP) : lo + ju - nA;
+      const T *krow = (pooled ? pk : kc) + (size_t)j * p.dim;
       float part = 0.f;
       if (shared_rows) {
 #pragma unroll
@@ -279,7 +410,7 @@ __global__ void __launch_bounds__(128) window_attn_kernel(const WindowAttn p) {
           part = fmaf(qv[i], vv[u][i], part);
         }
       } else {
-        const T *vrow = vc + (size_t)j * p.vdim;
+        const T *vrow = (pooled ? pv : vc) + (size_t)j * p.vdim;
 #pragma unroll
         for (int i = 0; i < NR; i++) {
           const int c = lane + 32 * i;
@@ -292,6 +423,7 @@ __global__ void __launch_bounds__(128) window_attn_kernel(const WindowAttn p) {
 #pragma unroll
     for (int u = 0; u < 4; u++) {
       s[u] = warp_sum(s[u]);
+      if (p.softcap > 0.f) s[u] = p.softcap * tanhf(s[u] / p.softcap);
       if (jj + u >= k1) s[u] = -INFINITY;
     }
     const float mn = fmaxf(fmaxf(mx, fmaxf(s[0], s[1])), fmaxf(s[2], s[3]));
@@ -331,8 +463,8 @@ __global__ void __launch_bounds__(128) window_attn_kernel(const WindowAttn p) {
     return;
   }
   float sink_term = 0.f;
-  if (p.sink) {
-    const float sk = DT<T>::to_f(reinterpret_cast<const T *>(p.sink)[h]);
+  if (p.sink || p.sink_zero) {
+    const float sk = p.sink ? DT<T>::to_f(reinterpret_cast<const T *>(p.sink)[h]) : 0.f;
     M4 = fmaxf(M4, sk);
     sink_term = expf(sk - M4);
   }
@@ -341,7 +473,7 @@ __global__ void __launch_bounds__(128) window_attn_kernel(const WindowAttn p) {
     f[w] = sm_m[w] == -INFINITY ? 0.f : expf(sm_m[w] - M4);
     L = fmaf(sm_l[w], f[w], L);
   }
-  const float il = 1.0f / (L + sink_term);
+  const float il = p.out_scale / (L + sink_term);
   const T *gate = reinterpret_cast<const T *>(p.gate);
   const float gh = gate && p.gate_per_head ? sigmoid_f(DT<T>::to_f(gate[(size_t)m * p.ldg + h])) : 1.f;
   T *out = reinterpret_cast<T *>(p.out) + (size_t)m * p.ldo + (size_t)h * p.vdim;
@@ -355,11 +487,11 @@ template <typename T>
 __global__ void __launch_bounds__(128) window_attn_merge_kernel(const WindowAttn p) {
   const int mh = blockIdx.x, m = mh / p.heads, h = mh % p.heads, stride = p.vdim + 2;
   const float *part = p.part + (size_t)mh * p.nsplit * stride;
-  float M = p.sink ? DT<T>::to_f(reinterpret_cast<const T *>(p.sink)[h]) : -INFINITY;
-  float L = p.sink ? 1.f : 0.f;  // the sink's term relative to its own logit; rescaled below
-  const float sk = M;
+  const bool sinks = p.sink || p.sink_zero;
+  const float sk = p.sink ? DT<T>::to_f(reinterpret_cast<const T *>(p.sink)[h]) : p.sink_zero ? 0.f : -INFINITY;
+  float M = sk, L;
   for (int s = 0; s < p.nsplit; s++) M = fmaxf(M, part[(size_t)s * stride]);
-  L = p.sink ? expf(sk - M) : 0.f;
+  L = sinks ? expf(sk - M) : 0.f;
   for (int s = 0; s < p.nsplit; s++) {
     const float ms = part[(size_t)s * stride];
     if (ms != -INFINITY) L = fmaf(part[(size_t)s * stride + 1], expf(ms - M), L);
@@ -373,14 +505,16 @@ __global__ void __launch_bounds__(128) window_attn_merge_kernel(const WindowAttn
       const float ms = part[(size_t)s * stride];
       if (ms != -INFINITY) a = fmaf(part[(size_t)s * stride + 2 + c], expf(ms - M), a);
     }
-    float o = a / L;
+    float o = a / L * p.out_scale;
     if (gate) o *= p.gate_per_head ? gh : sigmoid_f(DT<T>::to_f(gate[(size_t)m * p.ldg + (size_t)h * p.vdim + c]));
     out[c] = DT<T>::from_f(o);
   }
 }
 int window_attention(cudaStream_t st, int dtype, const WindowAttn &p, uint64_t *launches) {
   const int D = p.dim > p.vdim ? p.dim : p.vdim;
-  if (D > 32 * 24 || p.heads < 1 || p.kv_heads < 1 || p.heads % p.kv_heads || p.window < 0 || p.keep_first < 0) return (int)cudaErrorInvalidValue;
+  if (D > 32 * 24 || p.heads < 1 || p.kv_heads < 1 || p.heads % p.kv_heads || p.window < 0 || p.keep_first < 0 || p.chunk < 0 || p.pool < 0 ||
+      (p.pool > 0 && (!p.pk || !p.pv || (p.pos0 + p.S) / p.pool > p.pcap)))
+    return (int)cudaErrorInvalidValue;
   const bool split = p.part && p.nsplit > 1;
   const dim3 grid((unsigned)(p.B * p.S * p.heads), (unsigned)(split ? p.nsplit : 1));
   const size_t smem = (size_t)4 * p.vdim * sizeof(float);
@@ -397,7 +531,7 @@ int window_attention(cudaStream_t st, int dtype, const WindowAttn &p, uint64_t *
 
 // ---------------------------------------------------------------------------------------------- window attention, tiled
 // A CTA of four warps owns 64 consecutive rows of one (batch row, head); every warp 16 of them.  Keys come in tiles of 64: first
-// the kept first tokens that lie before the window of the block's first row, then the window up to the block's last row; the
+// the pooled blocks, then the kept first tokens that lie before the window of the block's first row, then the window up to the block's last row; the
 // visibility rule is applied per score, so a tile may straddle any edge.  Scores are 16 x 8 x 16 tensor-core products of the
 // staged q and key tiles with fp32 accumulators; the running softmax is fp32 per row (a quad of lanes shares a row); the weights
 // enter the second product as w_hi + w_lo in D (about 16 mantissa bits), the values through transposing shared-memory loads.
@@ -453,16 +587,22 @@ __global__ void __launch_bounds__(128) window_attn_tiled_kernel(const WindowAttn
   for (int n = 0; n < NV; n++) o[n][0] = o[n][1] = o[n][2] = o[n][3] = 0.f;
   float mrow[2] = {-INFINITY, -INFINITY}, lrow[2] = {0.f, 0.f};
   const int row_pos[2] = {p0 + warp * 16 + gid, p0 + warp * 16 + gid + 8};
-  const int lo = p.window > 0 ? max(0, p0 - p.window + 1) : 0;
-  const int nA = min(p.keep_first, lo);
-  const int tilesA = (nA + WT_KEYS - 1) / WT_KEYS, tilesB = (p1 - lo + 1 + WT_KEYS - 1) / WT_KEYS;
+  const int row_seen[2] = {pooled_seen(row_pos[0], p.window, p.pool), pooled_seen(row_pos[1], p.window, p.pool)};
+  const int row_lo[2] = {first_seen(row_pos[0], p.window, p.chunk), first_seen(row_pos[1], p.window, p.chunk)};
+  const int lo = first_seen(p0, p.window, p.chunk);
+  const int nP = pooled_seen(p1, p.window, p.pool), nA = min(p.keep_first, lo);
+  const int tilesP = (nP + WT_KEYS - 1) / WT_KEYS;
+  const int tilesA = tilesP + (nA + WT_KEYS - 1) / WT_KEYS, tilesB = (p1 - lo + 1 + WT_KEYS - 1) / WT_KEYS;
+  const T *pk = p.pool > 0 ? reinterpret_cast<const T *>(p.pk) + ((size_t)b * p.kv_heads + g) * p.pcap * p.dim : nullptr;
+  const T *pv = p.pool > 0 ? reinterpret_cast<const T *>(p.pv) + ((size_t)b * p.kv_heads + g) * p.pcap * p.vdim : nullptr;
   for (int tl = 0; tl < tilesA + tilesB; tl++) {
-    const int j0 = tl < tilesA ? tl * WT_KEYS : lo + (tl - tilesA) * WT_KEYS;
-    const int jend = tl < tilesA ? nA : p1 + 1;            // keys of this tile: [j0, min(j0 + 64, jend))
+    const bool pooled = tl < tilesP;
+    const int j0 = pooled ? tl * WT_KEYS : tl < tilesA ? (tl - tilesP) * WT_KEYS : lo + (tl - tilesA) * WT_KEYS;
+    const int jend = pooled ? nP : tl < tilesA ? nA : p1 + 1;  // keys of this tile: [j0, min(j0 + 64, jend))
     const int nk = min(WT_KEYS, jend - j0);
     __syncthreads();                                        // the previous tile has been consumed
-    stage_tile<T, LDS, HD>(ks, kc + (size_t)j0 * p.dim, p.dim, nk, p.dim);
-    stage_tile<T, LDS, HD>(vs, vc + (size_t)j0 * p.vdim, p.vdim, nk, p.vdim);
+    stage_tile<T, LDS, HD>(ks, (pooled ? pk : kc) + (size_t)j0 * p.dim, p.dim, nk, p.dim);
+    stage_tile<T, LDS, HD>(vs, (pooled ? pv : vc) + (size_t)j0 * p.vdim, p.vdim, nk, p.vdim);
     __syncthreads();
     float sc[8][4];
 #pragma unroll
@@ -481,8 +621,10 @@ __global__ void __launch_bounds__(128) window_attn_tiled_kernel(const WindowAttn
 #pragma unroll
       for (int e = 0; e < 4; e++) {
         const int j = j0 + n * 8 + 2 * qd + (e & 1), i = row_pos[e >> 1];
-        const bool vis = j < jend && j <= i && (p.window == 0 || i - j < p.window || j < p.keep_first);
-        sc[n][e] = vis ? sc[n][e] * p.scale : -INFINITY;
+        const bool vis = pooled ? j < row_seen[e >> 1] : j < jend && j <= i && (j >= row_lo[e >> 1] || j < p.keep_first);
+        float v = sc[n][e] * p.scale;
+        if (p.softcap > 0.f) v = p.softcap * (1.0f - __fdividef(2.0f, __expf(v * (2.0f / p.softcap)) + 1.0f));
+        sc[n][e] = vis ? v : -INFINITY;
         mnew[e >> 1] = fmaxf(mnew[e >> 1], sc[n][e]);
       }
     float corr[2];
@@ -534,15 +676,15 @@ __global__ void __launch_bounds__(128) window_attn_tiled_kernel(const WindowAttn
     l += __shfl_xor_sync(0xffffffffu, l, 1);
     l += __shfl_xor_sync(0xffffffffu, l, 2);
     float m = mrow[r], f = 1.f;
-    if (p.sink) {
-      const float sk = DT<T>::to_f(reinterpret_cast<const T *>(p.sink)[h]);
+    if (p.sink || p.sink_zero) {
+      const float sk = p.sink ? DT<T>::to_f(reinterpret_cast<const T *>(p.sink)[h]) : 0.f;
       const float mt = fmaxf(m, sk);
       f = m == -INFINITY ? 0.f : expf(m - mt);
       l = l * f + expf(sk - mt);
     }
     const int row = warp * 16 + gid + 8 * r;
     if (row >= n_rows) continue;
-    const float il = f / l;
+    const float il = f / l * p.out_scale;
     const size_t mrow_idx = (size_t)b * p.S + r0 + row;
     const float gh = gate && p.gate_per_head ? sigmoid_f(DT<T>::to_f(gate[mrow_idx * p.ldg + h])) : 1.f;
     T *out = reinterpret_cast<T *>(p.out) + mrow_idx * p.ldo + (size_t)h * p.vdim;
@@ -570,7 +712,7 @@ bool window_attention_tiled_ok(int dtype, const WindowAttn &p) {
   }();
   const int D = p.dim > p.vdim ? p.dim : p.vdim;
   return !off && dtype != 2 && p.S >= 16 && D <= 128 && p.dim % 8 == 0 && p.vdim % 8 == 0 && p.ldq % 8 == 0 && p.ldo % 2 == 0 && p.heads % p.kv_heads == 0 &&
-         ((uintptr_t)p.q & 15) == 0 && ((uintptr_t)p.kc & 15) == 0 && ((uintptr_t)p.vc & 15) == 0 && ((uintptr_t)p.out & 3) == 0;
+         ((uintptr_t)p.q & 15) == 0 && ((uintptr_t)p.kc & 15) == 0 && ((uintptr_t)p.vc & 15) == 0 && (((uintptr_t)p.pk | (uintptr_t)p.pv) & 15) == 0 && ((uintptr_t)p.out & 3) == 0;
 }
 template <typename T, int HD> static cudaError_t launch_window_tiled(cudaStream_t st, const WindowAttn &p) {
   const size_t smem = (size_t)3 * 64 * (HD + 8) * sizeof(T);

@@ -456,6 +456,41 @@ def netolorn_block_tensors(vb, cfg: Config, index: int) -> Dict[str, object]:
     return out
 
 
+def mafosun_block_tensors(vb, cfg: Config, index: int):
+    """The tensors of layer ``index`` of a Mafosun checkpoint by the field names of ``cake_b200_mixer_tensors``: (main, side or None),
+    each checked against the shape its MixerSpec declares.  Names under ``l<i>.``: ``norm1`` and ``norm2`` (both behind their sublayer)
+    and ``mix.*``: an attention layer has ``q, k, v, q.norm, k.norm, o``; a parallel layer the same under ``left.`` and ``right.{q,k,v,g,o}``;
+    ``mlp.{gate,up,down}`` (dense) or ``mlp.{router, e<j>.*}``."""
+    sp, H, name = cfg.layers[index], cfg.hidden_size, cfg.layer_name(index)
+
+    def get(short, shape):
+        t = vb.get(f"{name}.{short}")
+        if t is None:
+            raise KeyError(f"tensor {name}.{short} not found")
+        if tuple(t.shape) != tuple(shape):
+            raise ValueError(f"shape mismatch for {name}.{short}, expected: {list(shape)}, got: {list(t.shape)}")
+        return t
+
+    p, side = "mix.", None
+    if sp.side is not None:
+        p, r, rq = "mix.left.", sp.side, sp.side.heads * sp.side.dim
+        side = dict(q=get("mix.right.q", (rq, H)), k=get("mix.right.k", (rq, H)), v=get("mix.right.v", (r.inner, H)), g=get("mix.right.g", (r.inner, H)),
+                    o=get("mix.right.o", (H, r.inner)))
+    main: Dict[str, object] = dict(q=get(p + "q", (sp.heads * sp.dim, H)), k=get(p + "k", (sp.n_kv * sp.dim, H)), v=get(p + "v", (sp.n_kv * sp.vdim, H)),
+                                   q_norm=get(p + "q.norm", (sp.dim,)), k_norm=get(p + "k.norm", (sp.dim,)), o=get(p + "o", (H, sp.inner)),
+                                   post1=get("norm1", (H,)))
+    mo = sp.moe
+    if sp.dense_ff:
+        main.update(ff_gate=get("mlp.gate", (sp.dense_ff, H)), ff_up=get("mlp.up", (sp.dense_ff, H)), ff_down=get("mlp.down", (H, sp.dense_ff)))
+    elif mo is not None:
+        main.update(router=get("mlp.router", (mo.experts, H)), e_gate=[get(f"mlp.e{j}.gate", (mo.ff, H)) for j in range(mo.experts)],
+                    e_up=[get(f"mlp.e{j}.up", (mo.ff, H)) for j in range(mo.experts)],
+                    e_down=[get(f"mlp.e{j}.down", (H, mo.ff)) for j in range(mo.experts)])
+    if sp.dense_ff or mo is not None:
+        main["post2"] = get("norm2", (H,))
+    return main, side
+
+
 def detect_model_prefix(index_path: str, configured: str) -> str:
     """cake/mod.rs:335-357: the text before the first ``.layers.0.`` key of the index wins over the configured prefix."""
     if not os.path.exists(index_path):

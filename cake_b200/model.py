@@ -324,13 +324,14 @@ def _mixer_struct(sp, views, ctx, keep):
     decay = (ctypes.c_float * max(1, len(sp.decay)))(*sp.decay)
     keep.append(decay)
     spec = CMixerSpec(MIXER_KINDS[sp.type], sp.heads, sp.dim, sp.vdim, sp.rot_dim, sp.kv_rank, sp.scale,
-                      CRotarySpec(r.dims, r.base, r.factor, r.fast, r.slow, r.original),
+                      CRotarySpec(r.dims, r.base, r.factor, r.fast, r.slow, r.original, int(r.interleaved), *(r.stretch or (0.0, 0.0, 0.0, 0.0))),
                       decay if sp.decay else None, sp.state, sp.groups, sp.conv, sp.norm_groups,
-                      CMoeSpec(mo.experts, mo.identity, mo.top, mo.scale, mo.ff, mo.shared_ff, mo.act, mo.limit, mo.shared_limit, int(mo.logit_bias))
+                      CMoeSpec(mo.experts, mo.identity, mo.top, mo.scale, mo.ff, mo.shared_ff, mo.act, mo.limit, mo.shared_limit, int(mo.logit_bias),
+                               mo.groups, mo.groups_keep, int(mo.plain_weights))
                       if mo else CMoeSpec(),
                       sp.kv_heads, sp.bias_rows, sp.bias_max, sp.gate_cap, sp.norm_offset, sp.canon_taps, sp.dense_ff, sp.dense_act,
                       sp.dense_limit, None, sp.window, sp.keep_first, int(sp.qk_unit), sp.q_rank, sp.norm_kind, (ctypes.c_float * 4)(*sp.norm_alpha),
-                      sp.side_dim, sp.side_col)
+                      sp.side_dim, sp.side_col, sp.pool, sp.chunk, sp.softcap, int(sp.sink_zero), int(sp.qk_norm), int(sp.v_unit), sp.branch_scale)
     return spec, CMixerTensors(**args)
 
 
@@ -376,8 +377,32 @@ class SquashBlock(MixerBlock):
         return cls(name, h, ctx)
 
 
+class OutputNormBlock(MixerBlock):
+    """A layer of a Mafosun model: a mixer-list block (``cake_b200_block_load_mixer``) whose sublayers read the stream itself and are
+    normed on their output only; attention with pooled blocks in front of its window, or chunked attention beside retention with one
+    output projection over both; a dense relu or a group-limited routed feed-forward."""
+
+    @classmethod
+    def load(cls, name: str, ctx: Context) -> "OutputNormBlock":
+        from .loader import mafosun_block_tensors
+        cfg = ctx.config
+        index = [cfg.layer_name(i) for i in range(len(cfg.layers))].index(name)
+        sp = cfg.layers[index]
+        main, side = mafosun_block_tensors(ctx.var_builder, cfg, index)
+        keep = []
+        spec, tens = _mixer_struct(sp, main, ctx, keep)
+        if side is not None:
+            sspec, stens = _mixer_struct(sp.side, side, ctx, keep)
+            keep += [sspec, stens]
+            spec.side, tens.side = ctypes.pointer(sspec), ctypes.pointer(stens)
+        h = c_void_p()
+        check(lib().cake_b200_block_load_mixer(ctx.h, index, byref(spec), byref(tens), byref(h)))
+        return cls(name, h, ctx)
+
+
 # Config.block_kind -> the Forwarder that loads and runs its layers
-BLOCK_CLASSES = {"nigenex": ListedBlock, "setodra": MixerBlock, "nuvarax": SandwichBlock, "netolorn": SquashBlock}
+BLOCK_CLASSES = {"nigenex": ListedBlock, "setodra": MixerBlock, "nuvarax": SandwichBlock, "netolorn": SquashBlock,
+                 "mafosun": OutputNormBlock}
 
 
 @dataclass
@@ -424,7 +449,7 @@ class TextModelBase:
         lnf = rms_norm_weight(get(n_norm, () if cfg.scalar_final_norm else (cfg.hidden_size,)), cfg)   # text_model.rs:186-192
         head = None if n_head is None else get(n_head, (cfg.vocab_size, cfg.hidden_size))
         check(lib().cake_b200_head_load(ctx.h, ptr(emb), ptr(lnf), ptr(head)))
-        tables = cfg.pair_embedding or cfg.learned_positions or cfg.final_norm_offset or cfg.token_side_dim or cfg.final_norm_kind
+        tables = cfg.pair_embedding or cfg.learned_positions or cfg.final_norm_offset or cfg.token_side_dim or cfg.final_norm_kind or cfg.embed_norm
         if tables:   # embeddings that depend on a token's place in its sequence; the final norm's gain offset or squashing form; the token inputs
             from .capi import CEmbedTables
             pe = cfg.pair_embedding
@@ -436,9 +461,10 @@ class TextModelBase:
             side = get("side.embed", (cfg.vocab_size, side_cols)) if cfg.token_side_dim else None
             fb = get(n_norm + ".b", (cfg.hidden_size,)) if cfg.final_norm_kind else None
             fa = float(get(n_norm + ".alpha", ()).to(torch.float32)) if cfg.final_norm_kind else 0.0
+            en = get("embed.norm", (cfg.hidden_size,)) if cfg.embed_norm else None
             et = CEmbedTables(ptr(big), pe["buckets"] + 1 if pe else 0, pe["mul_prev"] if pe else 0, pe["mul_cur"] if pe else 0,
                               ptr(pos), int(pos.shape[0]) if pos is not None else 0, float(cfg.final_norm_offset),
-                              ptr(side), side_cols, int(cfg.final_norm_kind), fa, ptr(fb))
+                              ptr(side), side_cols, int(cfg.final_norm_kind), fa, ptr(fb), ptr(en))
             check(lib().cake_b200_head_load_tables(ctx.h, byref(et)))
         blocks: List[Forwarder] = []
         loaded: Dict[int, Forwarder] = {}   # a layer of a looped range appears once per pass and is loaded once

@@ -340,3 +340,39 @@ def make_netolorn_checkpoint(cfg: Config, dtype: str = "bf16", seed: int = 1234,
         if sp.side_dim:
             sd[f"{p}.side.gate"], sd[f"{p}.side.proj"], sd[f"{p}.side.norm"] = rn(sp.side_dim, H, s=4 * std), rn(H, sp.side_dim, s=0.3), ru(H, lo=0.2, hi=0.6)
     return sd
+
+
+def make_mafosun_checkpoint(cfg: Config, dtype: str = "bf16", seed: int = 1234, device="cpu", std: float = 0.05, router_std: float = 0.5) -> dict:
+    """Random weights of a Mafosun model under the names its checkpoints use: ``embed``, ``embed.norm``, ``final.norm`` and per layer
+    ``l<i>.norm1 / norm2``, ``l<i>.mix.*`` and ``l<i>.mlp.*``."""
+    gen = torch.Generator(device=device)
+    gen.manual_seed(seed * 1000003 + 626263)
+    td, H = TORCH_DTYPES[dtype], cfg.hidden_size
+
+    def rn(*shape, s=std):
+        return (torch.randn(shape, generator=gen, device=device, dtype=torch.float32) * s).to(td)
+
+    def ru(*shape, lo=0.8, hi=1.2):
+        return (torch.rand(shape, generator=gen, device=device, dtype=torch.float32) * (hi - lo) + lo).to(td)
+
+    sd = {"embed": rn(cfg.vocab_size, H, s=1.0), "embed.norm": ru(H), "final.norm": ru(H)}
+    for i, sp in enumerate(cfg.layers):
+        p = cfg.layer_name(i)
+        m = p + (".mix.left" if sp.side is not None else ".mix")
+        sd[f"{p}.norm1"] = ru(H, lo=0.4, hi=0.8)
+        sd[f"{m}.q"], sd[f"{m}.k"], sd[f"{m}.v"] = rn(sp.heads * sp.dim, H, s=4 * std), rn(sp.n_kv * sp.dim, H, s=4 * std), rn(sp.n_kv * sp.vdim, H, s=4 * std)
+        sd[f"{m}.q.norm"], sd[f"{m}.k.norm"], sd[f"{m}.o"] = ru(sp.dim, lo=0.5, hi=1.5), ru(sp.dim, lo=0.5, hi=1.5), rn(H, sp.inner, s=4 * std)
+        if sp.side is not None:
+            r, n = sp.side, f"{p}.mix.right"
+            sd[f"{n}.q"], sd[f"{n}.k"] = rn(r.heads * r.dim, H, s=4 * std), rn(r.heads * r.dim, H, s=4 * std)
+            sd[f"{n}.v"], sd[f"{n}.g"], sd[f"{n}.o"] = rn(r.inner, H, s=4 * std), rn(r.inner, H, s=4 * std), rn(H, r.inner, s=4 * std)
+        mo = sp.moe
+        if sp.dense_ff or mo is not None:
+            sd[f"{p}.norm2"] = ru(H, lo=0.4, hi=0.8)
+        if sp.dense_ff:
+            sd[f"{p}.mlp.gate"], sd[f"{p}.mlp.up"], sd[f"{p}.mlp.down"] = rn(sp.dense_ff, H, s=4 * std), rn(sp.dense_ff, H, s=4 * std), rn(H, sp.dense_ff, s=4 * std)
+        elif mo is not None:
+            sd[f"{p}.mlp.router"] = rn(mo.experts, H, s=router_std)
+            for j in range(mo.experts):
+                sd[f"{p}.mlp.e{j}.gate"], sd[f"{p}.mlp.e{j}.up"], sd[f"{p}.mlp.e{j}.down"] = rn(mo.ff, H, s=4 * std), rn(mo.ff, H, s=4 * std), rn(H, mo.ff, s=4 * std)
+    return sd

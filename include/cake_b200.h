@@ -219,7 +219,11 @@ int cake_b200_block_load_spec(cake_b200_ctx *, int layer_idx, const cake_b200_la
  *                            divided by its root mean square (eps of the ctx); score = (q . k) * scale; row i sees key j <= i when
  *                            window == 0, i - j < window or j < keep_first; the softmax's denominator also holds exp(sink_h) (sink
  *                            [heads], no key, no value; NULL = none); the concatenated heads are multiplied by sigmoid(g h)
- *                            (g [heads * vdim, hidden]; NULL = none); then o.  K and V rows live in the cache.
+ *                            (g [heads * vdim, hidden]; NULL = none); then o.  K and V rows live in the cache.  Optional parts:
+ *                            qk_norm (normed with gains before the rotation), v_unit, softcap, sink_zero, chunk (floor(i / chunk)
+ *                            == floor(j / chunk)), and pool: with blocks of P = pool positions, block b (positions b P .. b P + P - 1)
+ *                            is one more key of the same softmax once b P + P - 1 <= i - window; its key and value are the means of
+ *                            the block's cached keys and values and live in the cache beside them.
  *   CAKE_B200_MIX_LATENT_WINDOW  latent attention without positions: c_q = rms(dq h) * dq_norm ([q_rank]), q = uq c_q ([heads * dim,
  *                            q_rank]); c = rms(dkv h) * dkv_norm ([kv_rank]) is the only cached row; per head k = uk c, v = uv c
  *                            (steps of a few rows in the absorbed form: the query goes through uk, the weighted latent through
@@ -240,11 +244,13 @@ int cake_b200_block_load_spec(cake_b200_ctx *, int layer_idx, const cake_b200_la
  *   post1, post2 an RMS norm of the mixer's / feed-forward's output before it is added to the stream
  *   canon_taps   >= 1: the mixer reads h + conv(h), a causal convolution over time per channel of the normed input (canon
  *                [hidden, canon_taps], last tap = the current token, no bias, fp32); its last canon_taps - 1 inputs live in the cache
+ *   norm1, norm2 NULL beside post1 / post2: the sublayer reads the stream itself, only its output is normed
  *   side         a second mixer that reads the same input: both outputs are RMS-normed over the width with plain gains
- *                (branch_norm of each mixer's tensors) and averaged; the side mixer's spec / tensors use the mixer fields only
+ *                (branch_norm of each mixer's tensors) and averaged, or, without branch_norm, added with the two branch_scale; the
+ *                side mixer's spec / tensors use the mixer fields only.  Retention may be the main or the side mixer too
  *   dense_ff     > 0: a dense gated feed-forward of that width instead of the routed one (ff_gate, ff_up [dense_ff, hidden],
  *                ff_down [hidden, dense_ff]); dense_act 0 silu(g) u, 1 tanh-gelu(g) u, 2: g' = min(g, dense_limit), u' = clamp(u,
- *                -dense_limit, dense_limit), g' sigmoid(1.702 g') (u' + 1) */
+ *                -dense_limit, dense_limit), g' sigmoid(1.702 g') (u' + 1), 3: max(g, 0) u */
 #define CAKE_B200_MIX_LATENT 1
 #define CAKE_B200_MIX_RETENTION 2
 #define CAKE_B200_MIX_STATE_SPACE 3
@@ -259,6 +265,11 @@ typedef struct cake_b200_rotary_spec {
   double yarn_factor;  /* 0 = plain */
   double yarn_fast, yarn_slow;
   int yarn_original;
+  int interleaved;     /* 1: entries (2i, 2i + 1) form pair i instead of (i, i + dims / 2) */
+  /* stretch_factor > 0: pair i with wavelength l = 2 pi / f_i keeps f_i when l < stretch_original / stretch_high, gets f_i / stretch_factor
+   * when l > stretch_original / stretch_low, in between (1 - s) f_i / stretch_factor + s f_i with s = (stretch_original / l - stretch_low) /
+   * (stretch_high - stretch_low) */
+  double stretch_factor, stretch_low, stretch_high, stretch_original;
 } cake_b200_rotary_spec;
 typedef struct cake_b200_moe_spec {
   int experts, identity, top;
@@ -267,6 +278,9 @@ typedef struct cake_b200_moe_spec {
   int act;             /* 0 silu, 1 tanh-gelu, 2 clamped (limit / shared_limit) */
   float limit, shared_limit;
   int logit_bias;
+  int groups, groups_keep; /* groups > 1: the experts form that many equal groups of neighbours; only experts of the groups_keep groups with
+                              the largest best score may be chosen */
+  int plain_weights;       /* 1: the weights are the chosen experts' scores (times scale), not renormalised */
 } cake_b200_moe_spec;
 typedef struct cake_b200_mixer_spec {
   int kind;
@@ -292,6 +306,14 @@ typedef struct cake_b200_mixer_spec {
   int norm_kind;
   float norm_alpha[4];
   int side_dim, side_col;
+  /* sink attention: */
+  int pool;               /* > 0 (with a window): blocks of that many positions in front of the window, one key and value each */
+  int chunk;              /* > 0: row i sees the keys of its own chunk of that many positions, counted from position 0 */
+  float softcap;          /* > 0: score <- softcap * tanh(score / softcap) */
+  int sink_zero;          /* 1: the denominator holds one more term exp(0) without a value */
+  int qk_norm;            /* 1: RMS norm of every q and k head with the gains q_norm / k_norm [dim], in front of the rotation */
+  int v_unit;             /* 1: every value head is divided by its root mean square before it is cached */
+  float branch_scale;     /* with a side mixer and without branch norms: y = branch_scale * main + side->branch_scale * side */
 } cake_b200_mixer_spec;
 typedef struct cake_b200_mixer_tensors {
   const void *norm1, *norm2;                 /* [hidden]; norm2 NULL without a feed-forward */
@@ -312,6 +334,7 @@ typedef struct cake_b200_mixer_tensors {
   const void *dq, *dq_norm, *uq;             /* windowed latent attention: [q_rank, hidden], [q_rank], [heads * dim, q_rank] */
   const void *norm1_b, *post1_b, *norm2_b, *post2_b;  /* norm_kind 1: [hidden] each */
   const void *side_gate, *side_proj, *side_norm;      /* side_dim > 0: [side_dim, hidden], [hidden, side_dim], [hidden] */
+  const void *q_norm, *k_norm;               /* qk_norm: [dim] each */
 } cake_b200_mixer_tensors;
 int cake_b200_block_load_mixer(cake_b200_ctx *, int layer_idx, const cake_b200_mixer_spec *, const cake_b200_mixer_tensors *,
                                cake_b200_block **out);
@@ -366,6 +389,7 @@ typedef struct cake_b200_embed_tables {
   int final_norm_kind;      /* 1: the final norm is tanh(final_alpha x) * ln_f + final_bias ([hidden]) */
   float final_alpha;
   const void *final_bias;
+  const void *embed_norm;   /* [hidden]: the stream starts with the RMS norm of the (scaled) token embedding times this gain, or NULL */
 } cake_b200_embed_tables;
 int cake_b200_head_load_tables(cake_b200_ctx *, const cake_b200_embed_tables *);
 int cake_b200_embed_at(cake_b200_ctx *, cake_b200_cache *, const uint32_t *ids_host, int batch, int seq, int index_pos, void *x_dev);

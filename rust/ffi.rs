@@ -129,6 +129,7 @@ pub struct cake_b200_embed_tables {
     pub final_norm_kind: c_int,
     pub final_alpha: f32,
     pub final_bias: *const c_void,
+    pub embed_norm: *const c_void,
 }
 
 /// `cake_b200_rotary_spec`, `cake_b200_moe_spec`, `cake_b200_mixer_spec`, `cake_b200_mixer_tensors` (include/cake_b200.h): a
@@ -141,6 +142,11 @@ pub struct cake_b200_rotary_spec {
     pub yarn_fast: f64,
     pub yarn_slow: f64,
     pub yarn_original: c_int,
+    pub interleaved: c_int,
+    pub stretch_factor: f64,
+    pub stretch_low: f64,
+    pub stretch_high: f64,
+    pub stretch_original: f64,
 }
 #[repr(C)]
 pub struct cake_b200_moe_spec {
@@ -154,6 +160,9 @@ pub struct cake_b200_moe_spec {
     pub limit: f32,
     pub shared_limit: f32,
     pub logit_bias: c_int,
+    pub groups: c_int,
+    pub groups_keep: c_int,
+    pub plain_weights: c_int,
 }
 #[repr(C)]
 pub struct cake_b200_mixer_spec {
@@ -191,6 +200,14 @@ pub struct cake_b200_mixer_spec {
     pub norm_alpha: [f32; 4],
     pub side_dim: c_int,
     pub side_col: c_int,
+    // sink attention with pooled blocks or chunks, soft cap, zero sink, gained norms; branches added with constant factors
+    pub pool: c_int,
+    pub chunk: c_int,
+    pub softcap: f32,
+    pub sink_zero: c_int,
+    pub qk_norm: c_int,
+    pub v_unit: c_int,
+    pub branch_scale: f32,
 }
 #[repr(C)]
 pub struct cake_b200_mixer_tensors {
@@ -255,6 +272,8 @@ pub struct cake_b200_mixer_tensors {
     pub side_gate: *const c_void,
     pub side_proj: *const c_void,
     pub side_norm: *const c_void,
+    pub q_norm: *const c_void,
+    pub k_norm: *const c_void,
 }
 
 /// `cake_b200_block_variant` (include/cake_b200.h): norm placement and per-layer attention mode of the OLMo2 / Gemma3 /
