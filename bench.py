@@ -11,6 +11,7 @@ Llama-3-8B bf16, bs=1, 2k context, layers sharded over N GPUs of one box (N=1 ->
     python bench.py --workload setodra [--sizes 1k,2k]            # the Setodra design beside the closest existing model
     python bench.py --workload nuvarax [--sizes 1k,2k]            # the Nuvarax design beside the closest existing model
     python bench.py --workload netolorn [--sizes 1k,2k]           # the Netolorn design beside the closest existing models
+    python bench.py --workload mafosun [--sizes 1k,2k]            # the Mafosun design beside the closest existing models
 
 A "step" is one decoded token: one pass of the hot path (embed -> blocks -> ln_f/lm_head/argmax) at batch 1.
 tok/s follows the reference's definition (master.rs:131-166): prefill excluded.  Prints ONE JSON line (rank 0).
@@ -1386,6 +1387,111 @@ def netolorn_leg(env: Env, sizes=("1k", "2k"), batch: int = 4, seq: int = 4096, 
             "peaks": {"tensor_tflops": pk["tc"], "hbm_gbs": pk["hbm"], "source": pk["src"]}, "sizes": out}
 
 
+MAFOSUN_SIZES = {  # layer sizes of real models (random weights): pooled-block attention, chunked attention beside retention
+    "1k": dict(width=1024, ff=4224, window=1024, pool=16, chunk=1024, att=dict(heads=8, kv_heads=2, dim=128, vdim=128),
+               ret=dict(heads=4, dim=128, vdim=128), moe=dict(experts=32, top=4, ff=704, groups=4, keep=2)),
+    "2k": dict(width=2048, ff=11264, window=1024, pool=16, chunk=1024, att=dict(heads=16, kv_heads=4, dim=128, vdim=128),
+               ret=dict(heads=8, dim=128, vdim=128), moe=dict(experts=64, top=6, ff=1408, groups=8, keep=4)),
+}
+
+
+def mafosun_leg(env: Env, sizes=("1k", "2k"), batch: int = 4, seq: int = 4096, ctx_len: int = 2048, steps: int = 32, reps: int = 3) -> dict:
+    """`--workload mafosun`: the Mafosun design (mixer-list blocks whose sublayers are normed on their output only) in three 4-layer
+    models per size, two of them beside the framework's closest existing model at equal width:
+      attention   4 x (grouped-query attention with a full rotation, gained q / k norms, a window with pooled blocks in front of it, soft
+                  cap, zero sink + dense relu feed-forward)  beside the Netolorn attention layer (window, kept tokens, sink, gate)
+      parallel    4 x (chunked attention beside retention + group-limited routed feed-forward)  beside four Setodra retention layers
+                  with a routed feed-forward of the same sizes (no attention in them)
+      mixed       attention + dense, attention + routed, parallel + dense, parallel + routed (the headline number; no counterpart)
+    all through TextModelBase / forward_batch.  Workload and timing as in the Setodra leg."""
+    import torch
+    from cake_b200.config import Config, MixerSpec, MoeSpec, RotarySpec
+    from cake_b200.synth import make_mafosun_checkpoint, make_mixer_checkpoint, make_netolorn_checkpoint
+    pk = peaks()
+    out, launches, vocab = {}, 0, 32768
+    mseq = max(seq, ctx_len + steps + 8)
+    for name in sizes:
+        z = MAFOSUN_SIZES[name]
+        W, ff, win, pool, chunk, a, rt, mo = z["width"], z["ff"], z["window"], z["pool"], z["chunk"], z["att"], z["ret"], z["moe"]
+        H, G, D, V = a["heads"], a["kv_heads"], a["dim"], a["vdim"]
+        dense_ff = {"kind": "dense", "ff": ff}
+        routed = {"kind": "moe", "router": {"experts": mo["experts"], "top": mo["top"], "groups": {"count": mo["groups"], "keep": mo["keep"]}},
+                  "expert": {"ff": mo["ff"]}}
+        heads = {"heads": H, "kv_heads": G, "dim": D, "vdim": V, "scale": D ** -0.5}
+        att = dict(heads, softcap=50.0, mask={"size": win, "pool": pool},
+                   rot={"dims": D, "base": 500000.0, "scaling": {"factor": 8.0, "low": 1.0, "high": 4.0, "original": 2048}})
+        decay = [1.0 - 2.0 ** -(5 + i * 5.0 / rt["heads"]) for i in range(rt["heads"])]
+        par = {"left": dict(heads, mask={"size": chunk}), "left_scale": 0.6, "right_scale": 0.5,
+               "right": dict(rt, decay=decay, rot={"dims": rt["dim"], "base": 10000.0})}
+        layer = lambda mixer, mlp: {"type": "attention" if mixer is att else "parallel", "mixer": mixer, "mlp": mlp}
+        orders = {"attention": [layer(att, dense_ff)] * 4, "parallel": [layer(par, routed)] * 4,
+                  "mixed": [layer(att, dense_ff), layer(att, routed), layer(par, dense_ff), layer(par, routed)]}
+        # algorithmic work per token: products [flops = bytes of weights read by one decoded token], attended keys, state updates, cache rows
+        keys_win = lambda S: sum(min(i + 1, win) for i in range(S))
+        keys_pool = lambda S: sum(max(0, (i - win + 1) // pool) for i in range(S))
+        keys_chunk = lambda S: sum(i % chunk + 1 for i in range(S))
+        lin_att = 2.0 * W * (H * D + G * (D + V) + H * V)
+        lin_ret = 2.0 * W * rt["heads"] * (2 * rt["dim"] + 3 * rt["vdim"])
+        lin_ff = {"dense": 2.0 * W * 3 * ff, "moe": 2.0 * W * 3 * mo["top"] * mo["ff"] + 2.0 * W * mo["experts"]}
+        state = 4.0 * rt["heads"] * rt["dim"] * rt["vdim"]
+        row = {"size": z}
+        for arch in ("attention", "attention_closest", "parallel", "parallel_closest", "mixed"):
+            if arch in orders:
+                order = orders[arch]
+                cfg = Config.from_hf({"architecture": "Mafosun", "width": W, "vocab": vocab, "norm": {"eps": 1e-6}, "layers": order})
+                sd = make_mafosun_checkpoint(cfg, "bf16", seed=5, device=env.dev, std=0.02)
+                n_att = sum(1 for L in order if L["type"] == "attention")
+                n_par = 4 - n_att
+                flop_tok = 4 * lin_att + n_par * lin_ret + sum(lin_ff[L["mlp"]["kind"]] for L in order)
+                att_flops = 2.0 * H * (D + V) * (n_att * (keys_win(seq) + keys_pool(seq)) + n_par * keys_chunk(seq)) + n_par * state * seq
+                rows = n_att * (min(win, ctx_len) + max(0, ctx_len - win) // pool) + n_par * (ctx_len % chunk + steps / 2)
+                dbytes = flop_tok + 2.0 * G * (D + V) * rows + n_par * 2.0 * state
+            elif arch == "attention_closest":
+                L = {"type": "attention", "mlp": dense_ff,
+                     "mixer": dict(heads, mask={"size": win, "keep_first": 4},
+                                   rot={"dims": D, "base": 10000.0, "scaling": {"factor": 8.0, "original": 2048, "fast": 32.0, "slow": 1.0}})}
+                cfg = Config.from_hf({"architecture": "Netolorn", "width": W, "vocab": vocab, "norm": {"eps": 1e-6}, "layers": [L] * 4})
+                sd = make_netolorn_checkpoint(cfg, "bf16", seed=5, device=env.dev, std=0.02)
+                flop_tok = 4 * (lin_att + 2.0 * W * H * V + lin_ff["dense"])
+                att_flops = 4 * 2.0 * H * (D + V) * keys_win(seq)
+                dbytes = flop_tok + 4 * 2.0 * G * (D + V) * min(win, ctx_len)
+            else:
+                m = MoeSpec(scale=2.5, experts=mo["experts"], identity=0, top=mo["top"], ff=mo["ff"], shared_ff=0)
+                spec = MixerSpec(type="retention", heads=rt["heads"], dim=rt["dim"], vdim=rt["vdim"], decay=decay, rot=RotarySpec(dims=rt["dim"], base=10000.0), moe=m)
+                cfg = Config(hidden_size=W, intermediate_size=0, vocab_size=vocab, num_hidden_layers=4, num_attention_heads=rt["heads"],
+                             num_key_value_heads=rt["heads"], rms_norm_eps=1e-6, head_dim=rt["vdim"], max_seq_len=mseq, block_kind="setodra", layers=[spec] * 4,
+                             model_prefix="", embed_scale=1.0)
+                sd = make_mixer_checkpoint(cfg, "bf16", seed=5, device=env.dev, std=0.02)
+                flop_tok = 4 * (lin_ret + lin_ff["moe"])
+                att_flops = 4 * state * seq
+                dbytes = flop_tok + 4 * 2.0 * state
+            cfg.max_seq_len = mseq
+            t = _time_listed_model(env, cfg, sd, batch, seq, ctx_len, steps, reps, mseq)
+            del sd
+            torch.cuda.empty_cache()
+            launches += t["launches"]
+            M, ms, dms = batch * seq, t["prefill"]["ms"], t["decode"]["ms_per_token"]
+            flops = flop_tok * M + batch * att_flops + 2.0 * batch * vocab * W
+            dbytes += 2.0 * vocab * W
+            row[arch] = {"prefill": {"tok_s": M / (ms / 1e3), "ms": ms, "tflops": flops / (ms * 1e-3) / 1e12,
+                                     "frac_of_tensor_peak": flops / (ms * 1e-3) / 1e12 / pk["tc"], "finite": t["prefill"]["finite"],
+                                     "launches": t["prefill"]["launches"]},
+                         "decode": {"tok_s": 1e3 / dms, "ms_per_token": dms, "gb_s": dbytes / (dms * 1e-3) / 1e9,
+                                    "frac_of_hbm_peak": dbytes / (dms * 1e-3) / 1e9 / pk["hbm"], "launches_per_token": t["decode"]["launches_per_token"],
+                                    "finite": t["decode"]["finite"]}}
+        for kind in ("attention", "parallel"):   # how far from the roofline each is, the new design over the closest model (1 = equally far)
+            row[kind + "_prefill_distance"] = row[kind + "_closest"]["prefill"]["frac_of_tensor_peak"] / row[kind]["prefill"]["frac_of_tensor_peak"]
+            row[kind + "_decode_distance"] = row[kind + "_closest"]["decode"]["frac_of_hbm_peak"] / row[kind]["decode"]["frac_of_hbm_peak"]
+        out[name] = row
+    head = out[sizes[-1]]
+    return {"metric": f"mafosun prefill tok/s (4 layers, width {head['size']['width']}, bf16, bs={batch} x {seq})", "value": head["mixed"]["prefill"]["tok_s"],
+            "unit": "tok/s", "ms_per_step": head["mixed"]["prefill"]["ms"], "steps": reps, "warmup": 1, "gpu_launches": int(launches),
+            "config": {"workload": f"Mafosun (attention / parallel / mixed layer orders) vs the Netolorn attention layer and the Setodra retention layer at equal width, "
+                                   f"4 layers, bf16, prefill bs={batch} x {seq}, decode bs=1 at {ctx_len} context x {steps} steps",
+                       "l2": "prefill activations / decode weights exceed L2"},
+            "peaks": {"tensor_tflops": pk["tc"], "hbm_gbs": pk["hbm"], "source": pk["src"]}, "sizes": out}
+
+
 # ------------------------------------------------------------------------------------------------
 def run_cuda(args):
     env = Env(args)
@@ -1421,12 +1527,13 @@ def run_cuda(args):
             line.update({"n_gpus": 1, "higher_is_better": True, "scaling": "strong", "vs_baseline": None, "dtype": "bf16", "data": "synthetic"})
             emit(line)
         return
-    if args.workload == "netolorn":
+    if args.workload in ("netolorn", "mafosun"):
         if rank == 0:
             if env.sampler:
                 env.sampler.start()
             sizes = tuple((args.sizes if args.sizes != "2k,4k,4k-hd64" else "1k,2k").split(","))
-            line = netolorn_leg(env, sizes=sizes, batch=args.pf_batch, seq=args.pf_seq, steps=max(4, min(args.steps, 64)))
+            leg = netolorn_leg if args.workload == "netolorn" else mafosun_leg
+            line = leg(env, sizes=sizes, batch=args.pf_batch, seq=args.pf_seq, steps=max(4, min(args.steps, 64)))
             line["clocks"] = env.sampler.stop() if env.sampler else None
             line.update({"n_gpus": 1, "higher_is_better": True, "scaling": "strong", "vs_baseline": None, "dtype": "bf16", "data": "synthetic"})
             emit(line)
@@ -1504,9 +1611,9 @@ def main():
     ap.add_argument("--warmup", type=int, default=8)
     ap.add_argument("--impl", default="cuda", choices=["cuda", "reference"])
     ap.add_argument("--model", default="8b", choices=["8b", "70b"])
-    ap.add_argument("--workload", default="decode", choices=["decode", "prefill", "nigenex", "setodra", "nuvarax", "netolorn"])
-    ap.add_argument("--pf-batch", type=int, default=4, help="--workload setodra / nuvarax / netolorn: batch rows of the prefill step")
-    ap.add_argument("--pf-seq", type=int, default=4096, help="--workload setodra / nuvarax / netolorn: tokens per row of the prefill step")
+    ap.add_argument("--workload", default="decode", choices=["decode", "prefill", "nigenex", "setodra", "nuvarax", "netolorn", "mafosun"])
+    ap.add_argument("--pf-batch", type=int, default=4, help="--workload setodra / nuvarax / netolorn / mafosun: batch rows of the prefill step")
+    ap.add_argument("--pf-seq", type=int, default=4096, help="--workload setodra / nuvarax / netolorn / mafosun: tokens per row of the prefill step")
     ap.add_argument("--sizes", default="2k,4k,4k-hd64", help="--workload nigenex: which of NIGENEX_SIZES to run")
     ap.add_argument("--extras", default="auto", choices=["auto", "none", "all"],
                     help="auto: config0 + config4 at N=1, config3 (70B) at N=8; none: the headline only")

@@ -80,7 +80,8 @@ def close(got, want, dtype, what="", bar=None):
         assert e.max() < TOL[dtype], f"{what}: worst {e.max():.3g} at position {int(e.argmax())}"
     else:   # a router's close call may flip under 16-bit rounding
         bar = bar or TOL[dtype]
-        assert np.quantile(e, 0.95) < bar and e.max() < 6 * bar, f"{what}: 95 % within {np.quantile(e, 0.95):.3g}, worst {e.max():.3g} (bar {bar:.3g})"
+        assert np.quantile(e, 0.9) < bar and np.median(e) < bar / 2 and e.max() < max(6 * bar, 1.0), \
+            f"{what}: median {np.median(e):.3g}, 90 % within {np.quantile(e, 0.9):.3g}, worst {e.max():.3g} (bar {bar:.3g})"
 
 
 def plain(cfg, sd, toks, streams=None, fault=None):
@@ -517,20 +518,26 @@ def test_tiled_attention_of_other_head_sizes():
 
 @pytest.mark.gpu
 def test_a_far_block_carries_weight():
-    """One early block whose keys match the late queries: 400 positions back it still decides the row, through its mean.  Without
-    blocks the plain model's logits move by many tolerances; whole, in portions and decoded (over more than 256 visible keys the
-    split-key kernels run)."""
-    cfg = make_config([attn(heads=2, kv_heads=2, dim=16, vdim=16, size=40, pool=2, scale=3.0, softcap=60.0, rot=4, base=1e6, scaling=None, mlp=None),
+    """Queries of one token match the keys of another that fills one early block: 400 positions back it still decides the row, through
+    its mean.  Without that block's token the plain model's logits move by many tolerances; whole, in portions and decoded (over more
+    than 256 visible keys the split-key kernels run)."""
+    cfg = make_config([attn(heads=2, kv_heads=2, dim=16, vdim=16, size=40, pool=2, scale=1.0, softcap=60.0, rot=4, base=1e6, scaling=None, mlp=None),
                        par(size=300, scale=1.5, mlp=None)])
     sd = make_mafosun_checkpoint(cfg, "f32", seed=43)
-    sd["l0.mix.q"] = sd["l0.mix.k"].clone()        # a token's query matches the keys of the same token elsewhere
-    toks = tokens(460, cfg.vocab_size, seed=10)
-    toks[20:22] = [7, 7]                           # a block of one rare token ...
-    toks = [t if t != 7 or i in (20, 21, 455, 456) else 8 for i, t in enumerate(toks)]
-    toks[455], toks[456] = 7, 7                    # ... asked for again more than 400 positions later
+    ask, answer = 7, 9
+    sd["embed.norm"] = torch.ones_like(sd["embed.norm"])
+    e = P.rms_unit(sd["embed"], 1e-5)
+    u = (e[ask] - e[answer]) / (e[ask] - e[answer]).norm()
+    sd["l0.mix.q"] = sd["l0.mix.k"] @ (torch.eye(44) - 2 * u[:, None] * u[None, :])     # swaps the two embeddings, then looks for keys
+    sd["l0.mix.q.norm"] = sd["l0.mix.k.norm"].clone()
+    toks = [t if t not in (ask, answer) else 8 for t in tokens(460, cfg.vocab_size, seed=10)]
+    toks[20] = toks[21] = answer
+    toks[455] = toks[456] = ask
     want = plain(cfg, sd, toks)
+    other = list(toks)
+    other[20] = other[21] = 3
+    assert errors(plain(cfg, sd, other), want)[[455, 456]].min() > 50 * TOL["f32"]      # the far block decides these rows
     show_faults(cfg, sd, toks, want, ("no pool", "no chunk"), 50 * TOL["f32"])
-    assert errors(plain(cfg, sd, toks, fault="no pool"), want)[456] > 50 * TOL["f32"]
     r = Runner(cfg, sd, "f32")
     try:
         close(r.run("w", toks), want, "f32", "whole")
@@ -613,6 +620,20 @@ def test_other_sizes_and_tensor_core_shapes():
                 close(r.run("c", toks, cuts=[133, 2, 1, 150, 1]), whole, dtype, "portions against whole", bar)
         finally:
             r.close()
+    # without routers no position has an excuse: all of them within twice the worst that rounding the products causes
+    for L in layers:
+        L["mlp"] = dense(64)
+    cfg = make_config(layers, width=128, vocab=256)
+    sd = make_mafosun_checkpoint(cfg, "bf16", seed=53)
+    want = plain(cfg, sd, toks)
+    bar = 2 * errors(plain_with_rounded_products(cfg, sd, toks), want).max()
+    r = Runner(cfg, sd, "bf16")
+    try:
+        for cuts in (None, [133, 2, 1, 150, 1], [260] + [1] * 40):
+            e = errors(r.run("w", toks, cuts=cuts), want)
+            assert e.max() < bar, f"portions {cuts}: {e.max():.3g} at {int(e.argmax())} (bar {bar:.3g})"
+    finally:
+        r.close()
 
 
 @pytest.mark.gpu
