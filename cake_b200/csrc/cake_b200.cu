@@ -2069,7 +2069,7 @@ static int load_sub_mixer(cake_b200_ctx *c, cake_b200_block *b, const cake_b200_
 
 static int load_mixer_ext(cake_b200_ctx *c, int layer_idx, const cake_b200_mixer_spec *sp, const cake_b200_mixer_tensors *t, cake_b200_block **out) {
   // without norm1 / norm2 the sublayers read the stream itself and only their outputs are normed
-  const bool bare1 = !t->norm1, bare2 = !t->norm2;
+  const bool bare1 = !t->norm1, bare2 = !t->norm2 && (sp->dense_ff > 0 || sp->moe.experts + sp->moe.identity > 0);
   if ((bare1 && (!t->post1 || sp->canon_taps > 0 || sp->norm_kind != 0 || sp->norm_offset != 0.f)) || (bare2 && sp->norm_kind != 0))
     return fail(CAKE_B200_EINVAL, "layer %d: null norm1 needs post1, plain gains and no input convolution", layer_idx);
   const cake_b200_moe_spec &mo = sp->moe;

@@ -231,6 +231,16 @@ __global__ void __launch_bounds__(128) latent_attn_merge_kernel(const LatentAttn
   }
 }
 
+// four adjacent entries (8- / 16-byte load)
+template <typename T> __device__ __forceinline__ void load4(const T *s, float (&v)[4]) {
+  const uint2 u = *reinterpret_cast<const uint2 *>(s);
+  const float2 a = DT<T>::unpack2(u.x), b = DT<T>::unpack2(u.y);
+  v[0] = a.x; v[1] = a.y; v[2] = b.x; v[3] = b.y;
+}
+template <> __device__ __forceinline__ void load4<float>(const float *s, float (&v)[4]) {
+  const float4 u = *reinterpret_cast<const float4 *>(s);
+  v[0] = u.x; v[1] = u.y; v[2] = u.z; v[3] = u.w;
+}
 template <typename T> __device__ __forceinline__ void store4(T *d, const float (&v)[4]) {
 #pragma unroll
   for (int e = 0; e < 4; e++) d[e] = DT<T>::from_f(v[e]);
@@ -891,32 +901,33 @@ int gate_norm(cudaStream_t st, int dtype, const GateNorm &p, uint64_t *launches)
 
 // ---------------------------------------------------------------------------------------------- router
 constexpr int MOE_MAX_SLOTS = 8;  // experts + identity <= 256
-template <typename T>
+// NS: slots of 32 experts that a warp's lanes hold
+template <typename T, int NS>
 __global__ void __launch_bounds__(128) moe_router_kernel(const MoePlan p) {
   const int warp = (blockIdx.x * blockDim.x + threadIdx.x) >> 5, lane = threadIdx.x & 31;
   if (warp >= p.M) return;
   const int m = warp, E = p.experts + p.identity;
   const float *lg = p.logits + (size_t)m * p.ld;
   const T *corr = reinterpret_cast<const T *>(p.correction);
-  float z[MOE_MAX_SLOTS];
+  float z[NS];
 #pragma unroll
-  for (int sI = 0; sI < MOE_MAX_SLOTS; sI++) {
+  for (int sI = 0; sI < NS; sI++) {
     z[sI] = lane + 32 * sI < E ? lg[lane + 32 * sI] : -INFINITY;
     if (p.logit_bias && lane + 32 * sI < E) z[sI] += DT<T>::to_f(corr[lane + 32 * sI]);
   }
   float mx = -INFINITY;
 #pragma unroll
-  for (int sI = 0; sI < MOE_MAX_SLOTS; sI++) mx = fmaxf(mx, z[sI]);
+  for (int sI = 0; sI < NS; sI++) mx = fmaxf(mx, z[sI]);
   mx = warp_max(mx);
-  float sum = 0.f, sc[MOE_MAX_SLOTS], ch[MOE_MAX_SLOTS];
+  float sum = 0.f, sc[NS], ch[NS];
 #pragma unroll
-  for (int sI = 0; sI < MOE_MAX_SLOTS; sI++) {
+  for (int sI = 0; sI < NS; sI++) {
     sc[sI] = lane + 32 * sI < E ? expf(z[sI] - mx) : 0.f;
     sum += sc[sI];
   }
   sum = warp_sum(sum);
 #pragma unroll
-  for (int sI = 0; sI < MOE_MAX_SLOTS; sI++) {
+  for (int sI = 0; sI < NS; sI++) {
     const int e = lane + 32 * sI;
     if (p.logit_bias) {  // the choice is by the logits themselves; exp(z - max) / (sum over the chosen) is their softmax
       ch[sI] = z[sI];
@@ -926,43 +937,42 @@ __global__ void __launch_bounds__(128) moe_router_kernel(const MoePlan p) {
     ch[sI] = e < E ? sc[sI] + (corr ? DT<T>::to_f(corr[e]) : 0.f) : -INFINITY;
   }
   if (p.groups > 1) {  // lane g keeps the best score of group g (g = lane + 32 sI); the best groups_keep groups stay open
+    // (scores are not negative, so their bit patterns order like they do)
     const int gsz = E / p.groups;
-    float gb[MOE_MAX_SLOTS];
-    bool open[MOE_MAX_SLOTS];
+    unsigned gb[NS];
+    int grp[NS];
+    bool open[NS];
 #pragma unroll
-    for (int sI = 0; sI < MOE_MAX_SLOTS; sI++) { gb[sI] = -INFINITY; open[sI] = false; }
+    for (int sI = 0; sI < NS; sI++) { gb[sI] = 0u; open[sI] = false; grp[sI] = (lane + 32 * sI) / gsz; }
     for (int g = 0; g < p.groups; g++) {
-      float v = -INFINITY;
+      unsigned v = 0u;
 #pragma unroll
-      for (int sI = 0; sI < MOE_MAX_SLOTS; sI++) {
-        const int e = lane + 32 * sI;
-        if (e < E && e / gsz == g) v = fmaxf(v, sc[sI]);
-      }
-      v = warp_max(v);
+      for (int sI = 0; sI < NS; sI++)
+        if (grp[sI] == g) v = max(v, __float_as_uint(sc[sI]));   // lanes past the last expert belong to no group
+      v = __reduce_max_sync(0xffffffffu, v);
 #pragma unroll
-      for (int sI = 0; sI < MOE_MAX_SLOTS; sI++)
-        if (lane + 32 * sI == g) gb[sI] = v;
+      for (int sI = 0; sI < NS; sI++)
+        if (lane + 32 * sI == g) gb[sI] = v + 1u;                // 0 = no group, or taken
     }
     for (int k = 0; k < p.groups_keep; k++) {
-      float best = -INFINITY;
-      int bi = 0x7fffffff;
+      unsigned best = 0u;
 #pragma unroll
-      for (int sI = 0; sI < MOE_MAX_SLOTS; sI++)
-        if (gb[sI] > best) { best = gb[sI]; bi = lane + 32 * sI; }
+      for (int sI = 0; sI < NS; sI++) best = max(best, gb[sI]);
+      best = __reduce_max_sync(0xffffffffu, best);
+      int bi = -1;                                               // the first group with that score
 #pragma unroll
-      for (int o = 16; o > 0; o >>= 1) {
-        const float ob = __shfl_xor_sync(0xffffffffu, best, o);
-        const int oi = __shfl_xor_sync(0xffffffffu, bi, o);
-        if (ob > best || (ob == best && oi < bi)) { best = ob; bi = oi; }
+      for (int sI = 0; sI < NS; sI++) {
+        const unsigned who = __ballot_sync(0xffffffffu, gb[sI] == best);
+        if (bi < 0 && who) bi = 32 * sI + __ffs(who) - 1;
       }
 #pragma unroll
-      for (int sI = 0; sI < MOE_MAX_SLOTS; sI++) {
-        if (lane + 32 * sI == bi) gb[sI] = -INFINITY;
-        if ((lane + 32 * sI) / gsz == bi) open[sI] = true;
+      for (int sI = 0; sI < NS; sI++) {
+        if (lane + 32 * sI == bi) gb[sI] = 0u;
+        if (grp[sI] == bi) open[sI] = true;
       }
     }
 #pragma unroll
-    for (int sI = 0; sI < MOE_MAX_SLOTS; sI++)
+    for (int sI = 0; sI < NS; sI++)
       if (!open[sI]) ch[sI] = -INFINITY;
   }
   float wsum = 0.f, mine = 0.f;  // lane k keeps the score of the k-th choice
@@ -971,7 +981,7 @@ __global__ void __launch_bounds__(128) moe_router_kernel(const MoePlan p) {
     float best = -INFINITY, bs = 0.f;
     int bi = 0x7fffffff;
 #pragma unroll
-    for (int sI = 0; sI < MOE_MAX_SLOTS; sI++)
+    for (int sI = 0; sI < NS; sI++)
       if (ch[sI] > best) { best = ch[sI]; bi = lane + 32 * sI; bs = sc[sI]; }
 #pragma unroll
     for (int o = 16; o > 0; o >>= 1) {
@@ -980,7 +990,7 @@ __global__ void __launch_bounds__(128) moe_router_kernel(const MoePlan p) {
       if (ob > best || (ob == best && oi < bi)) { best = ob; bi = oi; bs = os; }
     }
 #pragma unroll
-    for (int sI = 0; sI < MOE_MAX_SLOTS; sI++)
+    for (int sI = 0; sI < NS; sI++)
       if (bi == lane + 32 * sI) ch[sI] = -INFINITY;
     wsum += bs;
     if (lane == k) { mine = bs; mine_id = bi; }
@@ -1067,7 +1077,14 @@ int moe_route(cudaStream_t st, int dtype, const MoePlan &p, uint64_t *launches) 
                        p.top > p.groups_keep * (p.experts / p.groups)))
     return (int)cudaErrorInvalidValue;
   if (p.logit_bias && !p.correction) return (int)cudaErrorInvalidValue;
-  MX_DISPATCH(dtype, (moe_router_kernel<T><<<(p.M + 3) / 4, 128, 0, st>>>(p)));
+  const int slots = (p.experts + p.identity + 31) / 32;
+  MX_DISPATCH(dtype, {
+    const unsigned grid = (unsigned)((p.M + 3) / 4);
+    if (slots <= 1) moe_router_kernel<T, 1><<<grid, 128, 0, st>>>(p);
+    else if (slots <= 2) moe_router_kernel<T, 2><<<grid, 128, 0, st>>>(p);
+    else if (slots <= 4) moe_router_kernel<T, 4><<<grid, 128, 0, st>>>(p);
+    else moe_router_kernel<T, MOE_MAX_SLOTS><<<grid, 128, 0, st>>>(p);
+  });
   int n = 1;
   if (p.experts > 0 && p.M * p.top <= MOE_SMALL_PAIRS) {
     moe_plan_small_kernel<<<1, 256, 0, st>>>(p);
@@ -2348,10 +2365,49 @@ __global__ void __launch_bounds__(256) embed_norm_kernel(const T *__restrict__ E
   const float inv = 1.0f / sqrtf(ss / (float)W + eps);
   for (int i = threadIdx.x; i < W; i += blockDim.x) out[i] = DT<T>::to_f(row[i]) * scale * inv * DT<T>::to_f(w[i]);
 }
+// widths that are multiples of four up to 8192: the row stays in registers between its sum of squares and its way out
+template <typename T, int NV>
+__global__ void __launch_bounds__(256) embed_norm_vec_kernel(const T *__restrict__ E, const uint32_t *__restrict__ ids, const T *__restrict__ w,
+                                                             float *__restrict__ x, int W, float scale, float eps) {
+  __shared__ float red[64];
+  const T *row = E + (size_t)ids[blockIdx.x] * W;
+  float4 *out = reinterpret_cast<float4 *>(x + (size_t)blockIdx.x * W);
+  float v[NV][4], ss = 0.f, z = 0.f;
+#pragma unroll
+  for (int q = 0; q < NV; q++) {
+    const int i = 4 * (threadIdx.x + 256 * q);
+    v[q][0] = v[q][1] = v[q][2] = v[q][3] = 0.f;
+    if (i < W) load4<T>(row + i, v[q]);
+#pragma unroll
+    for (int e = 0; e < 4; e++) {
+      v[q][e] *= scale;
+      ss = fmaf(v[q][e], v[q][e], ss);
+    }
+  }
+  block_sum2(ss, z, red);
+  const float inv = 1.0f / sqrtf(ss / (float)W + eps);
+#pragma unroll
+  for (int q = 0; q < NV; q++) {
+    const int i = 4 * (threadIdx.x + 256 * q);
+    if (i >= W) continue;
+    float g[4];
+    load4<T>(w + i, g);
+    out[i / 4] = make_float4(v[q][0] * inv * g[0], v[q][1] * inv * g[1], v[q][2] * inv * g[2], v[q][3] * inv * g[3]);
+  }
+}
 int embed_norm(cudaStream_t st, int dtype, const void *E, const uint32_t *ids, const void *w, float *x, int M, int W, int vocab, float scale, float eps,
                uint64_t *launches) {
   if (M < 1 || W < 1 || vocab < 1 || !E || !ids || !w || !x) return (int)cudaErrorInvalidValue;
-  MX_DISPATCH(dtype, (embed_norm_kernel<T><<<M, 256, 0, st>>>(reinterpret_cast<const T *>(E), ids, reinterpret_cast<const T *>(w), x, W, scale != 0.f ? scale : 1.f, eps)));
+  const float sc = scale != 0.f ? scale : 1.f;
+  const bool vec = W % 4 == 0 && W <= 8192 && (((uintptr_t)E | (uintptr_t)w | (uintptr_t)x) & 15) == 0;
+  MX_DISPATCH(dtype, {
+    const T *e = reinterpret_cast<const T *>(E), *g = reinterpret_cast<const T *>(w);
+    if (!vec) embed_norm_kernel<T><<<M, 256, 0, st>>>(e, ids, g, x, W, sc, eps);
+    else if (W <= 1024) embed_norm_vec_kernel<T, 1><<<M, 256, 0, st>>>(e, ids, g, x, W, sc, eps);
+    else if (W <= 2048) embed_norm_vec_kernel<T, 2><<<M, 256, 0, st>>>(e, ids, g, x, W, sc, eps);
+    else if (W <= 4096) embed_norm_vec_kernel<T, 4><<<M, 256, 0, st>>>(e, ids, g, x, W, sc, eps);
+    else embed_norm_vec_kernel<T, 8><<<M, 256, 0, st>>>(e, ids, g, x, W, sc, eps);
+  });
   MX_DONE(1);
 }
 

@@ -537,6 +537,7 @@ class TextModelBase:
             rows = int_array([int(w) for w in want])
             logits = ctx.empty(len(want), ctx.config.vocab_size, dtype=torch.float32)
             check(lib().cake_b200_logits_rows(ctx.h, ptr(x), b * s, rows, len(want), ptr(logits)))
+            torch.cuda.current_stream(ctx.device).wait_stream(ctx.torch_stream)   # a caller may read them on its own stream
             return logits
         logits = ctx.empty(b, ctx.config.vocab_size, dtype=ctx.logits_dtype)
         check(lib().cake_b200_logits(ctx.h, ptr(x), b, s, ptr(logits), None))
