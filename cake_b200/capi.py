@@ -106,7 +106,8 @@ class CRotarySpec(ctypes.Structure):
 class CMoeSpec(ctypes.Structure):
     """``cake_b200_moe_spec`` (include/cake_b200.h)."""
     _fields_ = [("experts", c_int), ("identity", c_int), ("top", c_int), ("scale", c_float), ("ff", c_int), ("shared_ff", c_int), ("act", c_int),
-                ("limit", c_float), ("shared_limit", c_float), ("logit_bias", c_int), ("groups", c_int), ("groups_keep", c_int), ("plain_weights", c_int)]
+                ("limit", c_float), ("shared_limit", c_float), ("logit_bias", c_int), ("groups", c_int), ("groups_keep", c_int), ("plain_weights", c_int),
+                ("sigmoid_scores", c_int), ("weigh_input", c_int)]
 
 
 class CMixerSpec(ctypes.Structure):
@@ -120,7 +121,8 @@ CMixerSpec._fields_ = [("kind", c_int), ("heads", c_int), ("dim", c_int), ("vdim
                        ("canon_taps", c_int), ("dense_ff", c_int), ("dense_act", c_int), ("dense_limit", c_float), ("side", POINTER(CMixerSpec)),
                        ("window", c_int), ("keep_first", c_int), ("qk_unit", c_int), ("q_rank", c_int), ("norm_kind", c_int), ("norm_alpha", c_float * 4),
                        ("side_dim", c_int), ("side_col", c_int), ("pool", c_int), ("chunk", c_int), ("softcap", c_float), ("sink_zero", c_int),
-                       ("qk_norm", c_int), ("v_unit", c_int), ("branch_scale", c_float)]
+                       ("qk_norm", c_int), ("v_unit", c_int), ("branch_scale", c_float), ("kv_back", c_int), ("decay_rank", c_int), ("decay_tau", c_float),
+                       ("streams", c_int), ("residual_mult", c_float)]
 
 
 MIXER_TENSOR_FIELDS = ("norm1", "norm2", "q", "k", "v", "g", "o", "dkv", "dkv_norm", "uk", "uv", "in", "conv", "conv_b", "dt_bias", "a_log", "d",
@@ -136,7 +138,7 @@ class CMixerTensors(ctypes.Structure):
 
 # fields behind `side` in the C struct (the newer mechanisms)
 MIXER_TENSOR_FIELDS_2 = ("sink", "dq", "dq_norm", "uq", "norm1_b", "post1_b", "norm2_b", "post2_b", "side_gate", "side_proj", "side_norm",
-                         "q_norm", "k_norm")
+                         "q_norm", "k_norm", "a1", "a2", "a2_b", "hc1_in", "hc1_out", "hc1_mix", "hc2_in", "hc2_out", "hc2_mix")
 CMixerTensors._fields_ = [(n, POINTER(_VP) if n.startswith("e_") else _VP) for n in MIXER_TENSOR_FIELDS] + [("side", POINTER(CMixerTensors))] + \
                          [(n, _VP) for n in MIXER_TENSOR_FIELDS_2]
 

@@ -73,12 +73,12 @@ class RotarySpec:
         return r
 
     @staticmethod
-    def from_dict(d: Optional[dict]) -> "RotarySpec":
+    def from_dict(d: Optional[dict], interleaved: bool = False) -> "RotarySpec":
         if not d:
-            return RotarySpec()
+            return RotarySpec(interleaved=interleaved)
         sc = d.get("scaling") or {}
         return RotarySpec(dims=int(d["dims"]), base=float(d["base"]), factor=float(sc.get("factor") or 0.0), fast=float(sc.get("fast") or 0.0),
-                          slow=float(sc.get("slow") or 0.0), original=int(sc.get("original") or 0))
+                          slow=float(sc.get("slow") or 0.0), original=int(sc.get("original") or 0), interleaved=interleaved)
 
     def to_dict(self) -> Optional[dict]:
         if not self.dims:
@@ -108,10 +108,12 @@ class MoeSpec:
     groups: int = 0          # > 1: equal groups of neighbouring experts; only those of the ``groups_keep`` groups with the best score may be chosen
     groups_keep: int = 0
     plain_weights: bool = False  # the weights are the chosen experts' scores, not renormalised
+    sigmoid_scores: bool = False  # scores are sigmoid(logit) instead of a softmax over all experts
+    weigh_input: bool = False    # a chosen expert reads weight * h; its output is added as it is
 
 
 MIXER_KINDS = {"latent_attention": 1, "retention": 2, "mamba2": 3, "delta": 4, "talking_attention": 5, "matrix_memory": 6,
-               "sink_attention": 7, "latent_window": 8}
+               "sink_attention": 7, "latent_window": 8, "gated_linear": 9}
 
 
 @dataclass
@@ -167,6 +169,15 @@ class MixerSpec:
     v_unit: bool = False
     branch_scale: float = 0.0
     pre_norms: bool = True
+    # sink_attention: one norm over the whole q (k) projection, keys and values of the layer ``kv_back`` layers earlier; gated_linear (linear
+    # attention with a decay per key channel from a low-rank product); several residual streams; a dense feed-forward without a gate
+    qk_norm_wide: bool = False
+    kv_back: int = 0
+    decay_tau: float = 0.0
+    decay_rank: int = 0      # rows of the first factor (read from the tensor's shape at load)
+    streams: int = 0
+    residual_mult: float = 1.0
+    dense_plain: bool = False
 
     @property
     def inner(self) -> int:
@@ -217,6 +228,12 @@ class Config:
     token_side_dim: int = 0           # > 0: a per-layer token input of that width (table `side.embed` [vocab, layers * dim])
     final_norm_kind: int = 0          # 1: the final norm is the squashing norm
     embed_norm: bool = False          # the stream starts with an RMS norm of the token embedding (gain `embed.norm`)
+    streams: int = 0                  # > 0: a token has that many residual streams side by side; the head reads their sum
+
+    @property
+    def stream_width(self) -> int:
+        """Elements of an activation row between blocks."""
+        return self.hidden_size * max(1, self.streams)
 
     def layer_variant(self, i: int, max_seq: Optional[int] = None) -> dict:
         """Norm placement and attention mode of layer ``i``, as the reference's per-architecture block.rs sets them up:
@@ -248,7 +265,7 @@ class Config:
     @property
     def layer_list(self) -> bool:
         """The checkpoint's config lists its layers one by one; such models keep an fp32 residual stream."""
-        return self.block_kind in ("nigenex", "setodra", "nuvarax", "netolorn", "mafosun")
+        return self.block_kind in ("nigenex", "setodra", "nuvarax", "netolorn", "mafosun", "lilenex")
 
     @property
     def scalar_final_norm(self) -> bool:
@@ -535,6 +552,81 @@ class Config:
                       head_dim=specs[0].vdim, max_seq_len=int(max_seq), block_kind="mafosun", layers=specs, model_prefix="",
                       loop_injects=False, tie_word_embeddings=True, embed_norm=True)
 
+    @staticmethod
+    def _from_lilenex(d: dict, max_seq: int = 4096) -> "Config":
+        """Lilenex ``config.json``: ``width``, ``vocab``, ``norm.eps``, ``streams``, ``residual_mult`` and ``layers``, whose entries give ``type``
+        (``attention``: grouped-query attention with ``rot`` (dims, base, scaling), ``mask`` (size, keep_first), ``scale`` and optionally
+        ``kv_from``, the layer whose keys and values it reads; ``gla``: gated linear attention with ``tau``), the mixer's sizes and the
+        feed-forward (``mlp``: kind ``dense`` with ``ff``; kind ``moe`` with ``router`` (experts, top), ``expert.ff`` and an optional ``shared.ff``;
+        or null).  The output projection is the embedding table.  Without ``streams`` the stream is one and sublayers add to it."""
+        streams, mult = int(d.get("streams") or 1), d.get("residual_mult")
+        specs = []
+        for i, L in enumerate(d["layers"]):
+            kind, m = L.get("type"), L["mixer"]
+            if kind == "attention":
+                mask, src = m.get("mask") or {}, m.get("kv_from")
+                size = int(mask.get("size") or 0)
+                sp = MixerSpec(type="sink_attention", heads=int(m["heads"]), kv_heads=int(m.get("kv_heads") or m["heads"]), dim=int(m["dim"]),
+                               vdim=int(m.get("vdim") or m["dim"]), scale=float(m["scale"]), rot=RotarySpec.from_dict(m.get("rot"), True), window=size,
+                               keep_first=int(mask.get("keep_first") or 0) if size else 0, qk_norm=True, qk_norm_wide=True,
+                               kv_back=0 if src is None else i - int(src))
+                if sp.rot.dims % 2 or sp.rot.dims > sp.dim:
+                    raise ValueError(f"layer {i}: rot.dims {sp.rot.dims} must be even and at most dim {sp.dim}")
+                if src is not None:
+                    o = specs[int(src)] if 0 <= int(src) < i else None
+                    if o is None or o.type != "sink_attention" or o.kv_back or (o.n_kv, o.dim, o.vdim) != (sp.n_kv, sp.dim, sp.vdim):
+                        raise ValueError(f"layer {i}: kv_from {src} is not an earlier attention layer with keys and values of these sizes")
+            elif kind == "gla":
+                sp = MixerSpec(type="gated_linear", heads=int(m["heads"]), dim=int(m["dim"]), vdim=int(m.get("vdim") or m["dim"]), decay_tau=float(m["tau"]))
+                if not sp.decay_tau > 0:
+                    raise ValueError(f"layer {i}: tau {sp.decay_tau}")
+            else:
+                raise ValueError(f"layer {i}: mixer type {kind!r} is not part of this design")
+            if sp.heads % sp.n_kv:
+                raise ValueError(f"layer {i}: {sp.heads} heads over {sp.n_kv} key heads")
+            mlp = L.get("mlp")
+            if mlp is not None:
+                if mlp.get("kind") == "dense":
+                    sp.dense_ff, sp.dense_act, sp.dense_plain = int(mlp["ff"]), 1, True
+                elif mlp.get("kind") == "moe":
+                    r, sh = mlp["router"], mlp.get("shared")
+                    sp.moe = MoeSpec(experts=int(r["experts"]), top=int(r["top"]), ff=int(mlp["expert"]["ff"]), shared_ff=int(sh["ff"]) if sh else 0,
+                                     plain_weights=True, sigmoid_scores=True, weigh_input=True)
+                    if not 1 <= sp.moe.top <= sp.moe.experts:
+                        raise ValueError(f"layer {i}: top {sp.moe.top} of {sp.moe.experts} experts")
+                else:
+                    raise ValueError(f"layer {i}: feed-forward kind {mlp.get('kind')!r} is not part of this design")
+            sp.streams, sp.residual_mult = streams, 1.0 if mult is None else float(mult)
+            specs.append(sp)
+        if not specs:
+            raise ValueError("config lists no layers")
+        return Config(hidden_size=int(d["width"]), intermediate_size=0, vocab_size=int(d["vocab"]), num_hidden_layers=len(specs),
+                      num_attention_heads=specs[0].heads, num_key_value_heads=specs[0].n_kv, rms_norm_eps=float(d["norm"]["eps"]),
+                      head_dim=specs[0].vdim, max_seq_len=int(max_seq), block_kind="lilenex", layers=specs, model_prefix="",
+                      loop_injects=False, tie_word_embeddings=True, streams=streams)
+
+    def to_lilenex(self) -> dict:
+        """The ``config.json`` of a Lilenex Config (inverse of ``_from_lilenex``)."""
+        layers = []
+        for i, s in enumerate(self.layers):
+            if s.type == "sink_attention":
+                kind, m = "attention", {"heads": s.heads, "kv_heads": s.n_kv, "dim": s.dim, "vdim": s.vdim, "scale": s.scale, "rot": s.rot.to_dict(),
+                                        "mask": {"size": s.window, "keep_first": s.keep_first} if s.window else None}
+                if s.kv_back:
+                    m["kv_from"] = i - s.kv_back
+            else:
+                kind, m = "gla", {"heads": s.heads, "dim": s.dim, "vdim": s.vdim, "tau": s.decay_tau}
+            mo = s.moe
+            if mo is not None:
+                mlp = {"kind": "moe", "router": {"experts": mo.experts, "top": mo.top}, "expert": {"ff": mo.ff}}
+                if mo.shared_ff:
+                    mlp["shared"] = {"ff": mo.shared_ff}
+            else:
+                mlp = {"kind": "dense", "ff": s.dense_ff} if s.dense_ff else None
+            layers.append({"type": kind, "mixer": m, "mlp": mlp})
+        return {"architecture": "Lilenex", "width": self.hidden_size, "vocab": self.vocab_size, "norm": {"eps": self.rms_norm_eps}, "streams": self.streams,
+                "residual_mult": self.layers[0].residual_mult, "layers": layers}
+
     def to_mafosun(self) -> dict:
         """The ``config.json`` of a Mafosun Config (inverse of ``_from_mafosun``)."""
         layers = []
@@ -641,6 +733,8 @@ class Config:
             return Config._from_netolorn(d)
         if d.get("architecture") == "Mafosun":
             return Config._from_mafosun(d)
+        if d.get("architecture") == "Lilenex":
+            return Config._from_lilenex(d)
         arch = Config.detect_arch(d)
         if arch in Config._OTHER_BLOCKS:
             raise ValueError(f"architecture {arch!r} is outside the block-forward path built here")
@@ -733,6 +827,8 @@ class Config:
             return self.to_netolorn()
         if self.block_kind == "mafosun":
             return self.to_mafosun()
+        if self.block_kind == "lilenex":
+            return self.to_lilenex()
         d = dict(
             architectures=[arch], hidden_size=self.hidden_size, intermediate_size=self.intermediate_size,
             vocab_size=self.vocab_size, num_hidden_layers=self.num_hidden_layers,
@@ -779,6 +875,7 @@ class CConfig(ctypes.Structure):
         ("sliding_window", ctypes.c_int), ("use_gelu_mlp", ctypes.c_int), ("embed_scale", ctypes.c_float),
         ("pre_reshape_qk_norm", ctypes.c_int),
         ("layer_list", ctypes.c_int), ("logit_softcap", ctypes.c_float), ("scalar_final_norm", ctypes.c_int),
+        ("streams", ctypes.c_int),
     ]
 
     @staticmethod
@@ -797,7 +894,7 @@ class CConfig(ctypes.Structure):
             rs.high_freq_factor if llama3 else 4.0, rs.original_max_position_embeddings if llama3 else 0,
             DTYPES[dtype],
             win, int(c.use_gelu_mlp), float(c.embed_scale or 0.0), int(c.pre_reshape_qk_norm),
-            int(c.layer_list), float(c.logit_softcap), int(c.scalar_final_norm),
+            int(c.layer_list), float(c.logit_softcap), int(c.scalar_final_norm), int(c.streams),
         )
 
 

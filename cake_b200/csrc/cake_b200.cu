@@ -243,7 +243,11 @@ struct cake_b200_block {
   void *m_sink = nullptr, *m_dq_norm = nullptr, *m_uq = nullptr;
   void *ln1_b = nullptr, *post1_b = nullptr, *ln2_b = nullptr, *post2_b = nullptr;
   void *sd_gate = nullptr, *sd_proj = nullptr, *sd_norm = nullptr;
-  void *m_qn = nullptr, *m_kn = nullptr;  // sink attention with qk_norm: gains [dim]
+  void *m_qn = nullptr, *m_kn = nullptr;  // sink attention with qk_norm: gains [dim], or of the whole projections
+  // gated linear attention: the second factor of the decays' low-rank product and its bias; several residual streams: the coefficients
+  // of both sublayers; a dense feed-forward without a gate; a shared expert without one
+  void *m_a2 = nullptr, *m_a2b = nullptr, *hc_in[2] = {nullptr, nullptr}, *hc_out[2] = {nullptr, nullptr}, *hc_mix[2] = {nullptr, nullptr};
+  bool ff_plain = false, shared_gated = false;
   // a side mixer that is added with constant factors: wo is [hidden, inner | side inner], one output projection for both
   bool joint = false;
   float out_scale = 1.f;
@@ -417,7 +421,7 @@ template <typename T> static int set_smem_attrs_T() {
   CU(cudaFuncSetAttribute(gemm_tc_kernel<T, EPI, 128>, cudaFuncAttributeMaxDynamicSharedMemorySize, TcCfg<128>::SMEM_BYTES));      \
   CU(cudaFuncSetAttribute(gemm_tc_kernel<T, EPI, 256>, cudaFuncAttributeMaxDynamicSharedMemorySize, TcCfg<256>::SMEM_BYTES));      \
   CU(cudaFuncSetAttribute(gemm_tc_kernel<T, EPI, 256, true>, cudaFuncAttributeMaxDynamicSharedMemorySize, TcCfg<256>::SMEM_BYTES));
-  SETT(TCE_PLAIN) SETT(TCE_RESIDUAL) SETT(TCE_SWIGLU) SETT(TCE_RESIDUAL_F32) SETT(TCE_SOFTCAP_F32)
+  SETT(TCE_PLAIN) SETT(TCE_RESIDUAL) SETT(TCE_SWIGLU) SETT(TCE_RESIDUAL_F32) SETT(TCE_SOFTCAP_F32) SETT(TCE_ACT)
   CU(cudaFuncSetAttribute(attn_window_tc_kernel<T>, cudaFuncAttributeMaxDynamicSharedMemorySize, FT_SMEM_BYTES));
   CU(cudaFuncSetAttribute(attn_window_tc_kernel<T>, cudaFuncAttributePreferredSharedMemoryCarveout, cudaSharedmemCarveoutMaxShared));
 #define SETW(HD) CU(cudaFuncSetAttribute(attn_window_mma_kernel<T, HD>, cudaFuncAttributeMaxDynamicSharedMemorySize, wm_smem_bytes<HD>()));
@@ -478,11 +482,14 @@ extern "C" int cake_b200_ctx_create(int device, const cake_b200_config *cfg, cak
     if (cfg->dtype != CAKE_B200_BF16 && cfg->dtype != CAKE_B200_F16 && cfg->dtype != CAKE_B200_F32)
       return fail(CAKE_B200_EINVAL, "dtype %d unsupported (bf16=0, f16=1, f32=2)", cfg->dtype);
     if (cfg->hidden < 1 || cfg->n_layers < 1 || cfg->vocab < 1 || cfg->max_seq < 1) return fail(CAKE_B200_EINVAL, "config dimensions must be positive");
+    if (cfg->streams < 0 || cfg->streams > mx::MAX_STREAMS || (cfg->streams > 0 && cfg->scalar_final_norm))
+      return fail(CAKE_B200_EINVAL, "%d residual streams (0..%d, and a vector gain of the final norm)", cfg->streams, mx::MAX_STREAMS);
     listed_cfg = *cfg;
     listed_cfg.inter = 64; listed_cfg.n_heads = 1; listed_cfg.n_kv_heads = 1; listed_cfg.head_dim = 16;
     listed_cfg.partial_rotary = 0.f; listed_cfg.rope_llama3 = 0; listed_cfg.sliding_window = 0;
     cfg = &listed_cfg;
   } else {
+  if (cfg->streams != 0) return fail(CAKE_B200_EINVAL, "several residual streams are for layer-list models");
   if (cfg->dtype != CAKE_B200_BF16 && cfg->dtype != CAKE_B200_F16)
     return fail(CAKE_B200_EINVAL, "dtype %d unsupported (bf16=0, f16=1; f32 is for layer-list models)", cfg->dtype);
   if (cfg->hidden < 1 || cfg->inter < 1 || cfg->n_heads < 1 || cfg->n_kv_heads < 1 || cfg->n_layers < 1 || cfg->vocab < 1 || cfg->max_seq < 1)
@@ -790,7 +797,8 @@ extern "C" void cake_b200_block_free(cake_b200_block *b) {
                   b->w_in, b->w_out, b->g, b->shift, b->r1, b->r2, b->m_dkv_norm, b->m_uk, b->m_uv, b->m_ukt, b->m_conv, b->m_conv_b, b->m_dt_bias,
                   b->m_a_log, b->m_d, b->m_norm, b->m_router, b->m_corr, b->m_eg, b->m_ed, b->m_cos, b->m_sin, b->m_decay,
                   b->post1, b->post2, b->canon, b->b_in, b->m_ob, b->m_talk, b->m_branch, b->m_ib, b->m_fb, b->m_bias,
-                  b->m_sink, b->m_dq_norm, b->m_uq, b->ln1_b, b->post1_b, b->ln2_b, b->post2_b, b->sd_gate, b->sd_proj, b->sd_norm, b->m_qn, b->m_kn};
+                  b->m_sink, b->m_dq_norm, b->m_uq, b->ln1_b, b->post1_b, b->ln2_b, b->post2_b, b->sd_gate, b->sd_proj, b->sd_norm, b->m_qn, b->m_kn,
+                  b->m_a2, b->m_a2b, b->hc_in[0], b->hc_in[1], b->hc_out[0], b->hc_out[1], b->hc_mix[0], b->hc_mix[1]};
   for (void *p : bufs)
     if (p) cudaFree(p);  // cudaFree synchronises with outstanding work
   if (b->side) cake_b200_block_free(b->side);
@@ -1424,7 +1432,7 @@ static int round_up(int v, int m) { return (v + m - 1) / m * m; }
 extern "C" int cake_b200_block_load_spec(cake_b200_ctx *c, int layer_idx, const cake_b200_layer_spec *sp,
                                          const cake_b200_layer_tensors *t, cake_b200_block **out) {
   if (!c || !sp || !t || !out) return fail(CAKE_B200_EINVAL, "null argument");
-  if (!c->cfg.layer_list) return fail(CAKE_B200_EINVAL, "block_load_spec needs a ctx created with layer_list = 1");
+  if (!c->cfg.layer_list || c->cfg.streams > 0) return fail(CAKE_B200_EINVAL, "block_load_spec needs a ctx created with layer_list = 1 and one residual stream");
   if (sp->heads < 1 || sp->kv_heads < 1 || sp->heads % sp->kv_heads || sp->head_dim < 1 || sp->head_dim > WA_MAX_HD)
     return fail(CAKE_B200_EINVAL, "layer %d: heads %d / kv_heads %d / head_dim %d unsupported (heads a multiple of kv_heads, head_dim <= %d)",
                 layer_idx, sp->heads, sp->kv_heads, sp->head_dim, WA_MAX_HD);
@@ -1521,7 +1529,7 @@ static int listed_gemm_tc(cake_b200_ctx *c, const void *A, const void *W, const 
   return gemm_tc_T<T, EPI>(c, A, W, nullptr, res, C, M, N, K, act, ldc, cap, x);
 }
 #define NO_TC_F32(EPI) template <> int listed_gemm_tc<float, EPI>(cake_b200_ctx *, const void *, const void *, const void *, void *, int, int, int, int, int, float, const TcExtra &) { return CAKE_B200_EINVAL; }
-NO_TC_F32(TCE_PLAIN) NO_TC_F32(TCE_SWIGLU) NO_TC_F32(TCE_RESIDUAL_F32) NO_TC_F32(TCE_SOFTCAP_F32)
+NO_TC_F32(TCE_PLAIN) NO_TC_F32(TCE_ACT) NO_TC_F32(TCE_SWIGLU) NO_TC_F32(TCE_RESIDUAL_F32) NO_TC_F32(TCE_SOFTCAP_F32)
 #undef NO_TC_F32
 
 // attention of a layer-list block: tensor cores for prompt portions in 16-bit D, the warp-split kernel for steps of a few
@@ -1746,7 +1754,8 @@ static int load_routed_ff(cake_b200_ctx *c, cake_b200_block *b, const cake_b200_
   CU(cudaMemsetAsync(b->m_router, 0, NP * H * es, 0));
   CU(cudaStreamSynchronize(0));
   RC(pipe_copy(c, b->m_router, Et * H * es, t->router, Et * H * es, Et * H * es, 1));
-  if (Is) RC(pipe_copy(c, (char *)b->m_router + Et * H * es, H * es, t->s_sg, H * es, H * es, 1));
+  b->shared_gated = Is && t->s_sg;
+  if (b->shared_gated) RC(pipe_copy(c, (char *)b->m_router + Et * H * es, H * es, t->s_sg, H * es, H * es, 1));
   if (t->correction) RC(upload(c, &b->m_corr, t->correction, Et * es));
   if (E) {
     // all experts stacked: gate / up row-interleaved per expert (as the dense blocks lay theirs out) and the down matrices,
@@ -1777,7 +1786,8 @@ extern "C" int cake_b200_block_load_mixer(cake_b200_ctx *c, int layer_idx, const
   if (!c || !sp || !t || !out) return fail(CAKE_B200_EINVAL, "null argument");
   if (!c->cfg.layer_list) return fail(CAKE_B200_EINVAL, "block_load_mixer needs a ctx created with layer_list = 1");
   if (mixer_kind_ext(sp->kind) || sp->side || sp->norm_offset != 0.f || sp->canon_taps > 0 || sp->dense_ff > 0 || t->post1 || t->post2 ||
-      sp->norm_kind != 0 || sp->side_dim > 0 || sp->moe.groups > 1 || sp->moe.plain_weights || sp->rot.interleaved)
+      sp->norm_kind != 0 || sp->side_dim > 0 || sp->moe.groups > 1 || sp->moe.plain_weights || sp->rot.interleaved ||
+      sp->streams > 0 || c->cfg.streams > 0 || sp->moe.sigmoid_scores || sp->moe.weigh_input || (sp->moe.shared_ff > 0 && !t->s_sg))
     return load_mixer_ext(c, layer_idx, sp, t, out);
   const cake_b200_moe_spec &mo = sp->moe;
   const bool has_ff = mo.experts + mo.identity > 0;
@@ -1874,7 +1884,7 @@ extern "C" int cake_b200_block_load_mixer(cake_b200_ctx *c, int layer_idx, const
 // convolution, a side mixer, a dense feed-forward) with the delta / talking-attention / matrix-memory mixers.
 static bool mixer_kind_ext(int kind) {
   return kind == CAKE_B200_MIX_DELTA || kind == CAKE_B200_MIX_TALKING_ATTENTION || kind == CAKE_B200_MIX_MATRIX_MEMORY ||
-         kind == CAKE_B200_MIX_SINK_ATTENTION || kind == CAKE_B200_MIX_LATENT_WINDOW;
+         kind == CAKE_B200_MIX_SINK_ATTENTION || kind == CAKE_B200_MIX_LATENT_WINDOW || kind == CAKE_B200_MIX_GATED_LINEAR;
 }
 static int sub_kv_heads(const cake_b200_mixer_spec &sp) { return sp.kv_heads > 0 ? sp.kv_heads : sp.heads; }
 
@@ -2007,24 +2017,28 @@ static int load_sub_mixer(cake_b200_ctx *c, cake_b200_block *b, const cake_b200_
     RC(upload(c, &b->m_fb, t->f_b, sp->heads * es));
     RC(upload(c, &b->m_norm, t->norm, inner * es));
   } else if (sp->kind == CAKE_B200_MIX_SINK_ATTENTION) {
-    if (!t->q || !t->k || !t->v || sp->window < 0 || sp->keep_first < 0 || sp->rot.dims > sp->dim)
-      return fail(CAKE_B200_EINVAL, "layer %d: sink attention needs q / k / v, window and keep_first >= 0 and an even rot.dims <= dim", layer_idx);
+    const bool shares = sp->kv_back > 0;  // keys and values are another layer's
+    if (!t->q || sp->kv_back < 0 || !t->k == !shares || !t->v == !shares || sp->window < 0 || sp->keep_first < 0 || sp->rot.dims > sp->dim)
+      return fail(CAKE_B200_EINVAL, "layer %d: sink attention needs q and k / v (or kv_back), window and keep_first >= 0 and an even rot.dims <= dim", layer_idx);
     if (std::max(sp->dim, sp->vdim) > 768) return fail(CAKE_B200_EINVAL, "layer %d: head sizes above 768", layer_idx);
     if (sp->pool < 0 || sp->chunk < 0 || sp->softcap < 0.f || (sp->pool > 0 && (sp->window < 1 || sp->chunk > 0 || sp->keep_first > 0)))
       return fail(CAKE_B200_EINVAL, "layer %d: pooled blocks need a window and stand beside neither chunks nor kept first tokens", layer_idx);
-    if (sp->qk_norm && (sp->qk_unit || !t->q_norm || !t->k_norm))
+    if (sp->qk_norm < 0 || sp->qk_norm > 2 || (sp->qk_norm && (sp->qk_unit || !t->q_norm || !t->k_norm != shares)) || (sp->qk_norm == 2 && sp->v_unit))
       return fail(CAKE_B200_EINVAL, "layer %d: qk_norm needs q_norm / k_norm and excludes qk_unit", layer_idx);
+    if (shares && (sp->pool > 0 || sp->v_unit)) return fail(CAKE_B200_EINVAL, "layer %d: shared keys and values are not built with pooled blocks or unit values", layer_idx);
     if (sp->sink_zero && t->sink) return fail(CAKE_B200_EINVAL, "layer %d: a learned sink and the zero sink exclude each other", layer_idx);
     if (sp->qk_norm) {
-      RC(upload(c, &b->m_qn, t->q_norm, (size_t)sp->dim * es));
-      RC(upload(c, &b->m_kn, t->k_norm, (size_t)sp->dim * es));
+      RC(upload(c, &b->m_qn, t->q_norm, (size_t)(sp->qk_norm == 2 ? sp->heads : 1) * sp->dim * es));
+      if (!shares) RC(upload(c, &b->m_kn, t->k_norm, (size_t)(sp->qk_norm == 2 ? G : 1) * sp->dim * es));
     }
     align8();
     b->pc[0] = add(t->q, (size_t)sp->heads * sp->dim, t->q_b);
-    align8();
-    b->pc[1] = add(t->k, (size_t)G * sp->dim, t->k_b);
-    align8();
-    b->pc[2] = add(t->v, (size_t)G * sp->vdim, t->v_b);
+    if (!shares) {
+      align8();
+      b->pc[1] = add(t->k, (size_t)G * sp->dim, t->k_b);
+      align8();
+      b->pc[2] = add(t->v, (size_t)G * sp->vdim, t->v_b);
+    }
     if (t->g) {
       align8();
       b->pc[3] = add(t->g, inner, nullptr);
@@ -2045,6 +2059,24 @@ static int load_sub_mixer(cake_b200_ctx *c, cake_b200_block *b, const cake_b200_
     b->pc[3] = add(t->g, inner, nullptr);
     RC(upload(c, (void **)&b->m_decay, sp->decay, sp->heads * sizeof(float)));
     RC(rope_tables());
+  } else if (sp->kind == CAKE_B200_MIX_GATED_LINEAR) {
+    if (!t->q || !t->k || !t->v || !t->g || !t->a1 || !t->a2 || !t->a2_b || !t->norm || sp->decay_rank < 1 || !(sp->decay_tau > 0.f) || G != sp->heads)
+      return fail(CAKE_B200_EINVAL, "layer %d: gated linear attention needs q / k / v / g / a1 / a2 / a2_b / norm, decay_rank >= 1, decay_tau > 0 and a key head per head", layer_idx);
+    if (sp->vdim > 1024) return fail(CAKE_B200_EINVAL, "layer %d: value heads above 1024", layer_idx);
+    const size_t qk = (size_t)sp->heads * sp->dim;
+    align8();
+    b->pc[0] = add(t->q, qk, nullptr);
+    align8();
+    b->pc[1] = add(t->k, qk, nullptr);
+    align8();
+    b->pc[2] = add(t->v, inner, nullptr);
+    align8();
+    b->pc[3] = add(t->g, inner, nullptr);
+    align8();
+    b->pc[4] = add(t->a1, (size_t)sp->decay_rank, nullptr);
+    RC(upload(c, &b->m_a2, t->a2, qk * sp->decay_rank * es));
+    RC(upload(c, &b->m_a2b, t->a2_b, qk * es));
+    RC(upload(c, &b->m_norm, t->norm, (size_t)sp->vdim * es));
   } else if (sp->kind == CAKE_B200_MIX_LATENT_WINDOW) {
     if (sp->q_rank < 1 || sp->kv_rank < 1 || sp->kv_rank > 768 || sp->window < 0 || sp->keep_first < 0 || !t->dq || !t->dq_norm || !t->uq || !t->dkv ||
         !t->dkv_norm || !t->uk || !t->uv)
@@ -2074,7 +2106,21 @@ static int load_mixer_ext(cake_b200_ctx *c, int layer_idx, const cake_b200_mixer
     return fail(CAKE_B200_EINVAL, "layer %d: null norm1 needs post1, plain gains and no input convolution", layer_idx);
   const cake_b200_moe_spec &mo = sp->moe;
   const bool has_moe = mo.experts + mo.identity > 0;
+  if (sp->streams != c->cfg.streams) return fail(CAKE_B200_EINVAL, "layer %d: %d residual streams in a ctx of %d", layer_idx, sp->streams, c->cfg.streams);
+  if (sp->streams > 0) {
+    const bool has_ff = has_moe || sp->dense_ff > 0;
+    if (sp->streams > mx::MAX_STREAMS || bare1 || bare2 || sp->side || sp->canon_taps > 0 || sp->norm_kind != 0 || sp->norm_offset != 0.f || sp->side_dim > 0 ||
+        t->post1 || t->post2 || t->o_b)
+      return fail(CAKE_B200_EINVAL, "layer %d: residual streams (at most %d) are built for pre-normed blocks without post norms, side mixers, input convolutions or token inputs",
+                  layer_idx, mx::MAX_STREAMS);
+    if (!t->hc1_in || !t->hc1_out || !t->hc1_mix || (has_ff && (!t->hc2_in || !t->hc2_out || !t->hc2_mix)))
+      return fail(CAKE_B200_EINVAL, "layer %d: residual streams need hc<q>_in / hc<q>_out / hc<q>_mix for every sublayer", layer_idx);
+  }
+  if (sp->kv_back > 0 && (sp->kind != CAKE_B200_MIX_SINK_ATTENTION || sp->side)) return fail(CAKE_B200_EINVAL, "layer %d: kv_back is for sink attention without a side mixer", layer_idx);
+  if (sp->side && sp->side->kv_back > 0) return fail(CAKE_B200_EINVAL, "layer %d: a side mixer has keys of its own", layer_idx);
   if (has_moe) {
+    if (mo.weigh_input && mo.identity > 0) return fail(CAKE_B200_EINVAL, "layer %d: weighted inputs are not built beside identity experts", layer_idx);
+    if (mo.sigmoid_scores && mo.logit_bias) return fail(CAKE_B200_EINVAL, "layer %d: sigmoid scores exclude a logit bias", layer_idx);
     if (sp->canon_taps > 0 || sp->norm_offset != 0.f || sp->dense_ff > 0)
       return fail(CAKE_B200_EINVAL, "layer %d: the routed feed-forward is not built beside an input convolution, offset gains or a dense feed-forward", layer_idx);
     if (mo.experts < 0 || mo.identity < 0 || mo.top < 1 || mo.top > mo.experts + mo.identity || mo.top > 32 || mo.experts + mo.identity > 256 ||
@@ -2083,7 +2129,7 @@ static int load_mixer_ext(cake_b200_ctx *c, int layer_idx, const cake_b200_mixer
                            mo.top > mo.groups_keep * (mo.experts / mo.groups))))
       return fail(CAKE_B200_EINVAL, "layer %d: bad router sizes (top <= 32, experts + identity <= 256) or null norm2 / router / correction", layer_idx);
     if (mo.experts > 0 && (!t->e_gate || !t->e_up || !t->e_down)) return fail(CAKE_B200_EINVAL, "layer %d: null expert table", layer_idx);
-    if (mo.shared_ff > 0 && (!t->s_gate || !t->s_up || !t->s_down || !t->s_sg)) return fail(CAKE_B200_EINVAL, "layer %d: null shared-expert pointer", layer_idx);
+    if (mo.shared_ff > 0 && (!t->s_gate || !t->s_up || !t->s_down)) return fail(CAKE_B200_EINVAL, "layer %d: null shared-expert pointer", layer_idx);
   }
   if (sp->norm_kind < 0 || sp->norm_kind > 1) return fail(CAKE_B200_EINVAL, "layer %d: norm_kind %d", layer_idx, sp->norm_kind);
   if (sp->norm_kind == 1) {
@@ -2101,8 +2147,8 @@ static int load_mixer_ext(cake_b200_ctx *c, int layer_idx, const cake_b200_mixer
   if (joint && (!scaled(sp->kind) || !scaled(sp->side->kind) || !t->o || !t->side->o))
     return fail(CAKE_B200_EINVAL, "layer %d: mixers added with constant factors are built for sink attention and retention", layer_idx);
   if (sp->canon_taps < 0 || (sp->canon_taps > 0 && !t->canon)) return fail(CAKE_B200_EINVAL, "layer %d: canon_taps %d without canon", layer_idx, sp->canon_taps);
-  if (sp->dense_ff < 0 || (sp->dense_ff > 0 && (!t->ff_gate || !t->ff_up || !t->ff_down || (bare2 && !t->post2) || sp->dense_act < 0 || sp->dense_act > 3)))
-    return fail(CAKE_B200_EINVAL, "layer %d: a dense feed-forward needs norm2 / ff_gate / ff_up / ff_down and dense_act in 0..3", layer_idx);
+  if (sp->dense_ff < 0 || (sp->dense_ff > 0 && (!t->ff_up || !t->ff_down || (bare2 && !t->post2) || sp->dense_act < 0 || sp->dense_act > 3 || (!t->ff_gate && sp->dense_act == 2))))
+    return fail(CAKE_B200_EINVAL, "layer %d: a dense feed-forward needs norm2 / ff_up / ff_down and dense_act in 0..3 (not 2 without ff_gate)", layer_idx);
   CU(cudaSetDevice(c->device));
   const size_t es = c->es, H = c->cfg.hidden;
   auto *b = new cake_b200_block{c, layer_idx, c->device};
@@ -2137,6 +2183,8 @@ static int load_mixer_ext(cake_b200_ctx *c, int layer_idx, const cake_b200_mixer
     for (int i = 0; i < 4; i++) b->ms.norm_alpha[i] = sp->norm_alpha[i];
     b->ms.side_dim = sp->side_dim;
     b->ms.side_col = sp->side_col;
+    b->ms.streams = sp->streams;
+    b->ms.residual_mult = sp->residual_mult;
     b->n_in = (int)row;
     b->n_in_pad = round_up(b->n_in, b->n_in > 1024 ? 256 : TC_BN);
     CU(cudaMalloc(&b->w_in, (size_t)b->n_in_pad * H * es + 16));
@@ -2161,10 +2209,23 @@ static int load_mixer_ext(cake_b200_ctx *c, int layer_idx, const cake_b200_mixer
       const size_t I = sp->dense_ff;
       if (t->norm2) RC(upload(c, &b->ln2, t->norm2, H * es));
       if (t->post2) RC(upload(c, &b->post2, t->post2, H * es));
-      CU(cudaMalloc(&b->wgu, 2 * I * H * es + 16));
-      RC(pipe_copy(c, b->wgu, 2 * H * es, t->ff_gate, H * es, H * es, I));
-      RC(pipe_copy(c, (char *)b->wgu + H * es, 2 * H * es, t->ff_up, H * es, H * es, I));
+      b->ff_plain = !t->ff_gate;
+      if (b->ff_plain) RC(upload(c, &b->wgu, t->ff_up, I * H * es));
+      else {
+        CU(cudaMalloc(&b->wgu, 2 * I * H * es + 16));
+        RC(pipe_copy(c, b->wgu, 2 * H * es, t->ff_gate, H * es, H * es, I));
+        RC(pipe_copy(c, (char *)b->wgu + H * es, 2 * H * es, t->ff_up, H * es, H * es, I));
+      }
       RC(upload(c, &b->wd, t->ff_down, H * I * es));
+    }
+    if (sp->streams > 0) {
+      const size_t n = sp->streams;
+      const void *src[2][3] = {{t->hc1_in, t->hc1_out, t->hc1_mix}, {t->hc2_in, t->hc2_out, t->hc2_mix}};
+      for (int q = 0; q < (has_moe || sp->dense_ff > 0 ? 2 : 1); q++) {
+        RC(upload(c, &b->hc_in[q], src[q][0], n * es));
+        RC(upload(c, &b->hc_out[q], src[q][1], n * es));
+        RC(upload(c, &b->hc_mix[q], src[q][2], n * n * es));
+      }
     }
     if (has_moe) {
       RC(load_routed_ff(c, b, mo, t, layer_idx));
@@ -2212,6 +2273,12 @@ static int cache_ensure_sub(cake_b200_cache *k, int slot, const cake_b200_block 
   const int G = sp.kv_heads, tag = sp.kind;
   const bool kv_rows = sp.kind == CAKE_B200_MIX_TALKING_ATTENTION || sp.kind == CAKE_B200_MIX_SINK_ATTENTION;
   const int width = kv_rows ? G * (sp.dim + sp.vdim) : sp.kind == CAKE_B200_MIX_LATENT_WINDOW ? sp.kv_rank : sp.heads * sp.dim * sp.vdim;
+  if (kv_rows && sp.kv_back > 0) {  // the rows of another layer: nothing of its own
+    const int src = slot - sp.kv_back;
+    if (src < 0 || k->kv_heads[src] != tag || k->kv_hd[src] != width || !k->k[src])
+      return fail(CAKE_B200_ESTATE, "cache entry %d shares the keys of entry %d, which holds none of that geometry", slot, src);
+    return CAKE_B200_OK;
+  }
   if (k->kv_heads[slot] && (k->kv_heads[slot] != tag || k->kv_hd[slot] != width))
     return fail(CAKE_B200_ESTATE, "cache entry %d was used with another layer geometry", slot);
   if (k->kv_heads[slot]) return CAKE_B200_OK;
@@ -2326,6 +2393,10 @@ template <typename Take> static SubScratch sub_scratch(const cake_b200_ctx *c, c
   }
   s.o32 = (float *)take(M * inner * sizeof(float));
   if (sp.kind == CAKE_B200_MIX_RETENTION) return s;
+  if (sp.kind == CAKE_B200_MIX_GATED_LINEAR) {
+    s.f1 = (float *)take(M * (size_t)sp.heads * sp.dim * sizeof(float));
+    return s;
+  }
   s.f1 = (float *)take(M * sp.heads * sizeof(float));
   s.f2 = (float *)take(M * sp.heads * sizeof(float));
   if (sp.kind == CAKE_B200_MIX_DELTA) {
@@ -2345,6 +2416,8 @@ static bool moe_on_tc(const cake_b200_ctx *c, const cake_b200_block *b);
 template <typename Take> static MoeScratch moe_scratch(const cake_b200_ctx *c, const cake_b200_block *b, size_t M, Take &&take);
 template <typename T>
 static int enqueue_routed_ff(cake_b200_ctx *c, const cake_b200_block *b, const MoeScratch &w, const void *h, const float *x, float *out, int M, uint64_t *lc);
+template <typename T>
+static int enqueue_shared_ff(cake_b200_ctx *c, const cake_b200_block *b, const MoeScratch &w, const void *h, const float *x, float *out, int M);
 struct ExtScratch {
   void *h, *proj, *act, *side;
   float *h32;
@@ -2443,8 +2516,11 @@ static int run_sub_mixer(cake_b200_ctx *c, const cake_b200_block *b, cake_b200_c
       MX(mx::talk_attention(st, dt, ta, lc));
     }
   } else if (sp.kind == CAKE_B200_MIX_SINK_ATTENTION) {
-    mx::QkPrep qp{proj, ldp, b->pc[0], b->pc[1], b->pc[2], b->m_cos, b->m_sin, sp.rot.dims, sp.qk_unit, c->cfg.rms_eps, w.qh, kc->k[slot], kc->v[slot],
-                  B, S, sp.heads, G, sp.dim, sp.vdim, kc->cap, pos0, sp.rot.interleaved, b->m_qn, b->m_kn, sp.v_unit};
+    const bool shares = sp.kv_back > 0;  // the step's rows of the shared keys and values are in the cache already
+    if (shares) slot -= sp.kv_back;
+    mx::QkPrep qp{proj, ldp, b->pc[0], b->pc[1], b->pc[2], b->m_cos, b->m_sin, sp.rot.dims, sp.qk_unit, c->cfg.rms_eps, w.qh,
+                  shares ? nullptr : kc->k[slot], shares ? nullptr : kc->v[slot], B, S, sp.heads, shares ? 0 : G, sp.dim, sp.vdim, kc->cap, pos0,
+                  sp.rot.interleaved, b->m_qn, b->m_kn, sp.v_unit, sp.qk_norm == 2};
     MX(mx::qk_prep(st, dt, qp, lc));
     const int pcap = sp.pool > 0 ? std::max(1, kc->cap / sp.pool) : 0;
     if (sp.pool > 0) {  // the blocks that this step completes
@@ -2466,6 +2542,14 @@ static int run_sub_mixer(cake_b200_ctx *c, const cake_b200_block *b, cake_b200_c
                      1.0f / sqrtf((float)sp.dim), b->m_cos, b->m_sin, sp.rot.dims, kc->rec_state[slot], w.o32, B, S, sp.heads, sp.dim, sp.vdim, pos0};
     MX(mx::recurrence(st, dt, r, lc));
     mx::GateNorm gn{w.o32, proj + b->pc[3], ldp, nullptr, w.att, M, inner, sp.heads, 0, c->cfg.rms_eps, 0, 0, nullptr, ldo, b->out_scale};
+    MX(mx::gate_norm(st, dt, gn, lc));
+  } else if (sp.kind == CAKE_B200_MIX_GATED_LINEAR) {
+    mx::ChannelDecay cd{proj + b->pc[4], ldp, sp.decay_rank, b->m_a2, b->m_a2b, w.f1, M, sp.heads * sp.dim, sp.decay_tau};
+    MX(mx::channel_decay(st, dt, cd, lc));
+    mx::Recurrence r{proj + b->pc[0], proj + b->pc[1], proj + b->pc[2], ldp, ldp, ldp, 1, nullptr, 0, nullptr, nullptr, nullptr, nullptr, 1.0f,
+                     nullptr, nullptr, 0, kc->rec_state[slot], w.o32, B, S, sp.heads, sp.dim, sp.vdim, pos0, nullptr, nullptr, w.f1, 1.0f / sqrtf((float)sp.dim)};
+    MX(mx::recurrence(st, dt, r, lc));
+    mx::GateNorm gn{w.o32, proj + b->pc[3], ldp, b->m_norm, w.att, M, inner, sp.heads, 0, c->cfg.rms_eps, 0, sp.vdim, nullptr, ldo};
     MX(mx::gate_norm(st, dt, gn, lc));
   } else if (sp.kind == CAKE_B200_MIX_LATENT_WINDOW) {
     // both latents are normed (the key / value latent straight into the cache), the query latent is expanded and taken through
@@ -2516,6 +2600,65 @@ static int run_sub_mixer(cake_b200_ctx *c, const cake_b200_block *b, cake_b200_c
     MX(mx::gate_norm(st, dt, gn, lc));
   }
   return with_out ? gemm_f32_out<T>(c, w.att, b->wo, w.y, M, H, inner) : CAKE_B200_OK;
+}
+
+// the dense feed-forward of an ext block on rows h [M, hidden] in D: y (fp32) = down(act(gate h) * (up h)), or down(act(up h)) without a gate
+template <typename T> static int enqueue_dense_ff(cake_b200_ctx *c, const cake_b200_block *b, const void *h, void *act, float *y, int M) {
+  const cake_b200_mixer_spec &sp = b->ms;
+  const int I = sp.dense_ff, H = c->cfg.hidden;
+  if (b->ff_plain) {
+    if (listed_tc<T>(c, M, I, H)) RC((listed_gemm_tc<T, TCE_ACT>(c, h, b->wgu, nullptr, act, M, I, H, sp.dense_act, I)));
+    else {
+      RowsGemm gu{h, b->wgu, nullptr, act, M, I, H, H, I, sp.dense_act, 0.f};
+      RC((gemm_rows_T<T, RE_ACT>(c, gu)));
+    }
+  } else if (listed_tc<T>(c, M, 2 * I, H)) RC((listed_gemm_tc<T, TCE_SWIGLU>(c, h, b->wgu, nullptr, act, M, 2 * I, H, sp.dense_act, I, sp.dense_limit)));
+  else {
+    RowsGemm gu{h, b->wgu, nullptr, act, M, 2 * I, H, H, I, sp.dense_act, sp.dense_limit};
+    RC((gemm_rows_T<T, RE_GATE_UP>(c, gu)));
+  }
+  return gemm_f32_out<T>(c, act, b->wd, y, M, H, I);
+}
+
+// one block with several residual streams: every sublayer reads norm(sum in X) and its output joins all streams in the kernel that
+// also reads out the next sublayer's input (of this block or of `next`, the block that runs behind it in the call); h_ready: the
+// scratch's first buffer, which every block of a step shares, holds this block's first input already.
+template <typename T>
+static int enqueue_streams_layer(cake_b200_ctx *c, const cake_b200_block *b, const cake_b200_block *next, int l, cake_b200_cache *kc, const float *cur, float *x_out,
+                                 int B, int S, int pos0, uint64_t *lc, bool &h_ready) {
+  const cake_b200_mixer_spec &sp = b->ms;
+  const int M = B * S, H = c->cfg.hidden, dt = c->cfg.dtype;
+  const ExtScratch w = ext_scratch(c, b, (size_t)M, (char *)c->mx_ws, S, pos0 + S);
+  auto mix = [&](const float *x, const float *a, const MoeScratch *mo, int q, const cake_b200_block *nb, int nq) -> int {
+    const bool wr = q >= 0;
+    mx::StreamMix sm{x, x_out, a, mo ? mo->y : nullptr, mo ? mo->ids : nullptr, mo ? mo->pos_of : nullptr, mo ? sp.moe.top : 0, mo ? sp.moe.experts : 0,
+                     wr ? b->hc_mix[q] : nullptr, wr ? b->hc_out[q] : nullptr, sp.residual_mult, nb ? nb->hc_in[nq] : nullptr,
+                     nb ? (nq ? nb->ln2 : nb->ln1) : nullptr, nb ? w.h : nullptr, M, H, sp.streams, c->cfg.rms_eps};
+    MX(mx::stream_mix(c->stream, dt, sm, lc));
+    return CAKE_B200_OK;
+  };
+  if (!h_ready) RC(mix(cur, nullptr, nullptr, -1, b, 0));
+  if (listed_tc<T>(c, M, b->n_in_pad, H)) RC(gemm_bias_tc<T>(c, w.h, b->w_in, b->b_in, w.proj, M, b->n_in_pad, H));
+  else {
+    RowsGemm gi{w.h, b->w_in, nullptr, w.proj, M, b->n_in, H, H, b->n_in_pad, 0, 0.f, nullptr, b->b_in};
+    RC((gemm_rows_T<T, RE_STORE>(c, gi)));
+  }
+  RC(run_sub_mixer<T>(c, b, kc, l, w.a, (const T *)w.proj, b->n_in_pad, B, S, pos0, lc, c->stream, true));
+  const bool has_moe = sp.moe.experts + sp.moe.identity > 0, has_ff = has_moe || sp.dense_ff > 0;
+  RC(mix(cur, w.a.y, nullptr, 0, has_ff ? b : next, has_ff ? 1 : 0));
+  if (has_moe && (!sp.moe.weigh_input || b->shared_gated)) {  // the slots' weighted sum is made first
+    RC(enqueue_routed_ff<T>(c, b, w.moe, w.h, nullptr, w.a.y, M, lc));
+    RC(mix(x_out, w.a.y, nullptr, 1, next, 0));
+  } else if (has_moe) {  // the experts' outputs are summed on their way into the streams (weighted inputs: every weight is one)
+    RC(enqueue_routed_ff<T>(c, b, w.moe, w.h, nullptr, nullptr, M, lc));
+    if (sp.moe.shared_ff) RC(enqueue_shared_ff<T>(c, b, w.moe, w.h, nullptr, w.a.y, M));
+    RC(mix(x_out, sp.moe.shared_ff ? w.a.y : nullptr, &w.moe, 1, next, 0));
+  } else if (has_ff) {
+    RC(enqueue_dense_ff<T>(c, b, w.h, w.act, w.a.y, M));
+    RC(mix(x_out, w.a.y, nullptr, 1, next, 0));
+  }
+  h_ready = next != nullptr;
+  return CAKE_B200_OK;
 }
 
 // one ext block: x_out = x + post1(mixers(canon(norm1(x)))), then x_out += post2(ff(norm2(x_out)))
@@ -2587,7 +2730,7 @@ static int enqueue_ext_layer(cake_b200_ctx *c, const cake_b200_block *b, int l, 
   // a sublayer that is normed on its output only: norm, residual sum and the next sublayer's operand in one pass
   const bool bare_ff = !b->ln2 && (sp.dense_ff > 0 || has_moe);
   auto merge = [&](const float *a, const void *post, const float *x, const MoeScratch *mo) -> int {
-    mx::StreamMerge sm{mo ? nullptr : a, mo ? mo->y : nullptr, mo ? mo->wts : nullptr, mo ? mo->ids : nullptr, mo ? mo->pos_of : nullptr,
+    mx::StreamMerge sm{mo ? nullptr : a, mo ? mo->y : nullptr, mo && !sp.moe.weigh_input ? mo->wts : nullptr, mo ? mo->ids : nullptr, mo ? mo->pos_of : nullptr,
                        mo ? sp.moe.top : 0, mo ? sp.moe.experts : 0, post, x, x_out, wide ? nullptr : w.h, M, H, eps};
     MX(mx::stream_merge(st, dt, sm, lc));
     x_in_h = !wide;
@@ -2636,13 +2779,7 @@ static int enqueue_ext_layer(cake_b200_ctx *c, const cake_b200_block *b, int l, 
     } else RC(enqueue_routed_ff<T>(c, b, w.moe, op, x_out, x_out, M, lc));
   }
   if (sp.dense_ff > 0) {
-    const int I = sp.dense_ff;
-    if (listed_tc<T>(c, M, 2 * I, H)) RC((listed_gemm_tc<T, TCE_SWIGLU>(c, op, b->wgu, nullptr, w.act, M, 2 * I, H, sp.dense_act, I, sp.dense_limit)));
-    else {
-      RowsGemm gu{op, b->wgu, nullptr, w.act, M, 2 * I, H, H, I, sp.dense_act, sp.dense_limit};
-      RC((gemm_rows_T<T, RE_GATE_UP>(c, gu)));
-    }
-    RC(gemm_f32_out<T>(c, w.act, b->wd, w.a.y, M, H, I));
+    RC(enqueue_dense_ff<T>(c, b, op, w.act, w.a.y, M));
     if (bare_ff) RC(merge(w.a.y, b->post2, x_out, nullptr));
     else if (squash && b->post2) {
       mx::TanhNorm p2{w.a.y, nullptr, 1, 0, b->post2, b->post2_b, sp.norm_alpha[3], x_out, x_out, nullptr, M, H};
@@ -2786,36 +2923,45 @@ static int enqueue_routed_ff(cake_b200_ctx *c, const cake_b200_block *b, const M
   RowsGemm gr{h, b->m_router, nullptr, w.logits, M, NP, H, H, NP, 0, 0.f};
   if (listed_tc<T>(c, M, NP, H)) RC((listed_gemm_tc<T, TCE_SOFTCAP_F32>(c, h, b->m_router, nullptr, w.logits, M, NP, H, 0, 0)));
   else RC((gemm_rows_T<T, RE_SOFTCAP_F32>(c, gr)));
-  mx::MoePlan mp{w.logits, NP, b->m_corr, mo.shared_ff ? 1 : 0, M, H, mo.experts, mo.identity, mo.top, mo.scale, w.ids, w.wts,
-                 w.sgate, w.tile, w.counts, w.perm, w.pos_of, w.tile_expert, w.max_tiles, mo.logit_bias, mo.groups, mo.groups_keep, mo.plain_weights};
+  mx::MoePlan mp{w.logits, NP, b->m_corr, b->shared_gated ? 1 : 0, M, H, mo.experts, mo.identity, mo.top, mo.scale, w.ids, w.wts,
+                 w.sgate, w.tile, w.counts, w.perm, w.pos_of, w.tile_expert, w.max_tiles, mo.logit_bias, mo.groups, mo.groups_keep, mo.plain_weights,
+                 mo.sigmoid_scores};
   MX(mx::moe_route(st, dt, mp, lc));
   if (mo.experts && w.sorted) {  // grouped products: sorted rows of h -> act(gate) * up -> down, expert e at row e * N of the stacked weights
     const int rows = w.max_tiles * w.tile;
-    MX(mx::moe_gather(st, dt, h, w.perm, w.sorted, rows, H, mo.top, lc));
+    MX(mx::moe_gather(st, dt, h, w.perm, w.sorted, rows, H, mo.top, lc, mo.weigh_input ? w.wts : nullptr));
     TcExtra xg;
     xg.tile_group = w.tile_expert;
     xg.n_groups = mo.experts;
     RC((listed_gemm_tc<T, TCE_SWIGLU>(c, w.sorted, b->m_eg, nullptr, w.act, rows, 2 * mo.ff, H, mo.act, mo.ff, mo.limit, xg)));
     RC((listed_gemm_tc<T, TCE_SOFTCAP_F32>(c, w.act, b->m_ed, nullptr, w.y, rows, H, mo.ff, 0, 0, 0.f, xg)));
   } else if (mo.experts) {
-    mx::MoeExperts me{h, b->m_eg, b->m_ed, w.act, w.y, M, H, mo.ff, mo.top, mo.act, w.perm, w.tile_expert, w.tile, w.max_tiles, mo.limit};
+    mx::MoeExperts me{h, b->m_eg, b->m_ed, w.act, w.y, M, H, mo.ff, mo.top, mo.act, w.perm, w.tile_expert, w.tile, w.max_tiles, mo.limit,
+                      mo.weigh_input ? w.wts : nullptr};
     MX(mx::moe_experts(st, dt, me, lc));
   }
   if (!out) return CAKE_B200_OK;  // the caller sums the sorted outputs itself
-  mx::MoeCombine mc{x, out, h, w.y, w.wts, w.ids, w.pos_of, M, H, mo.top, mo.experts};
+  mx::MoeCombine mc{x, out, h, w.y, mo.weigh_input ? nullptr : w.wts, w.ids, w.pos_of, M, H, mo.top, mo.experts};
   MX(mx::moe_combine(st, dt, mc, lc));
-  if (mo.shared_ff) {
-    RowsGemm gu{h, b->wgu, nullptr, w.sact, M, 2 * mo.shared_ff, H, H, mo.shared_ff, mo.act, mo.shared_limit};
-    if (listed_tc<T>(c, M, 2 * mo.shared_ff, H)) RC((listed_gemm_tc<T, TCE_SWIGLU>(c, h, b->wgu, nullptr, w.sact, M, 2 * mo.shared_ff, H, mo.act, mo.shared_ff, mo.shared_limit)));
-    else RC((gemm_rows_T<T, RE_GATE_UP>(c, gu)));
-    RowsGemm gd{w.sact, b->wd, out, out, M, H, mo.shared_ff, mo.shared_ff, H, 0, 0.f, w.sgate};
-    if (listed_tc<T>(c, M, H, mo.shared_ff) && ((uintptr_t)out & 15) == 0) {
-      TcExtra xs;
-      xs.row_scale = w.sgate;
-      RC((listed_gemm_tc<T, TCE_RESIDUAL_F32>(c, w.sact, b->wd, out, out, M, H, mo.shared_ff, 0, 0, 0.f, xs)));
-    } else RC((gemm_rows_T<T, RE_RESIDUAL_F32>(c, gd)));
+  return mo.shared_ff ? enqueue_shared_ff<T>(c, b, w, h, out, out, M) : CAKE_B200_OK;
+}
+// out = (x ? x : 0) + gate * shared expert(h), the gate sigmoid(s_sg . h) where the block has one; out may alias x
+template <typename T>
+static int enqueue_shared_ff(cake_b200_ctx *c, const cake_b200_block *b, const MoeScratch &w, const void *h, const float *x, float *out, int M) {
+  const cake_b200_moe_spec &mo = b->ms.moe;
+  const int H = c->cfg.hidden;
+  RowsGemm gu{h, b->wgu, nullptr, w.sact, M, 2 * mo.shared_ff, H, H, mo.shared_ff, mo.act, mo.shared_limit};
+  if (listed_tc<T>(c, M, 2 * mo.shared_ff, H)) RC((listed_gemm_tc<T, TCE_SWIGLU>(c, h, b->wgu, nullptr, w.sact, M, 2 * mo.shared_ff, H, mo.act, mo.shared_ff, mo.shared_limit)));
+  else RC((gemm_rows_T<T, RE_GATE_UP>(c, gu)));
+  if (!x) return b->shared_gated ? fail(CAKE_B200_EINVAL, "a gated shared expert needs the sum it joins") : gemm_f32_out<T>(c, w.sact, b->wd, out, M, H, mo.shared_ff);
+  const float *gate = b->shared_gated ? w.sgate : nullptr;
+  RowsGemm gd{w.sact, b->wd, x, out, M, H, mo.shared_ff, mo.shared_ff, H, 0, 0.f, gate};
+  if (listed_tc<T>(c, M, H, mo.shared_ff) && (((uintptr_t)out | (uintptr_t)x) & 15) == 0) {
+    TcExtra xs;
+    xs.row_scale = gate;
+    return listed_gemm_tc<T, TCE_RESIDUAL_F32>(c, w.sact, b->wd, x, out, M, H, mo.shared_ff, 0, 0, 0.f, xs);
   }
-  return CAKE_B200_OK;
+  return gemm_rows_T<T, RE_RESIDUAL_F32>(c, gd);
 }
 
 // x_in, x_out: [B, S, hidden] fp32 (may alias)
@@ -2848,6 +2994,11 @@ static int enqueue_mixer_layers(cake_b200_ctx *c, cake_b200_block *const *blocks
       const cake_b200_block *b = blocks[i];
       const cake_b200_mixer_spec &sp = b->ms;
       const int l = block_idx[i], inner = sp.heads * sp.vdim;
+      if (sp.streams > 0) {
+        RC(enqueue_streams_layer<T>(c, b, i + 1 < n ? blocks[i + 1] : nullptr, l, kc, cur, x_out, B, S, pos0, lc, x_in_h));
+        cur = x_out;
+        continue;
+      }
       if (b->ext) {
         RC(enqueue_ext_layer<T>(c, b, l, kc, cur, x_out, B, S, pos0, lc, x_in_h));
         cur = x_out;
@@ -2952,7 +3103,7 @@ static int enqueue_mixer_layers(cake_b200_ctx *c, cake_b200_block *const *blocks
 
 extern "C" int cake_b200_stream_inject(cake_b200_ctx *c, float *x_dev, const float *x0_dev, const void *vec, int slot, int rows) {
   if (!c || !x_dev || !vec || rows < 1 || slot < 0 || slot >= 64) return fail(CAKE_B200_EINVAL, "bad stream_inject arguments");
-  if (!c->cfg.layer_list) return fail(CAKE_B200_EINVAL, "stream_inject is for models with an fp32 residual stream");
+  if (!c->cfg.layer_list || c->cfg.streams > 0) return fail(CAKE_B200_EINVAL, "stream_inject is for models with one fp32 residual stream");
   CU(cudaSetDevice(c->device));
   if (c->inject_src[slot] != vec) {
     if (c->inject_vec[slot]) { CU(cudaStreamSynchronize(c->stream)); cudaFree(c->inject_vec[slot]); c->inject_vec[slot] = nullptr; }
@@ -2967,7 +3118,7 @@ extern "C" int cake_b200_stream_inject(cake_b200_ctx *c, float *x_dev, const flo
 
 extern "C" int cake_b200_stream_project(cake_b200_ctx *c, float *x_dev, const float *x0_dev, const void *w, int rows) {
   if (!c || !x_dev || !x0_dev || !w || rows < 1) return fail(CAKE_B200_EINVAL, "bad stream_project arguments");
-  if (!c->cfg.layer_list) return fail(CAKE_B200_EINVAL, "stream_project is for models with an fp32 residual stream");
+  if (!c->cfg.layer_list || c->cfg.streams > 0) return fail(CAKE_B200_EINVAL, "stream_project is for models with one fp32 residual stream");
   CU(cudaSetDevice(c->device));
   const size_t H = c->cfg.hidden;
   if (c->proj_src != w) {
@@ -3017,6 +3168,12 @@ extern "C" int cake_b200_forward_batch(cake_b200_ctx *c, cake_b200_block *const 
     if (kc->len[block_idx[i]] != index_pos)
       return fail(CAKE_B200_ESTATE, "block %d: index_pos %d != cache length %d (clear the cache or feed positions in order)",
                   block_idx[i], index_pos, kc->len[block_idx[i]]);
+    if (blocks[i]->mixer && blocks[i]->ms.kv_back > 0) {  // the layer it shares keys with ran these positions: earlier in this call or before it
+      const int src = block_idx[i] - blocks[i]->ms.kv_back;
+      bool ran = kc->len[src] == index_pos + seq;
+      for (int j = 0; j < i; j++) ran = ran || block_idx[j] == src;
+      if (!ran) return fail(CAKE_B200_ESTATE, "block %d shares the keys of block %d, which has not run this step's positions", block_idx[i], src);
+    }
   }
   if (mixer) {  // fp32 residual stream
     RC(enqueue_mixer_layers(c, blocks, block_idx, n_blocks, kc, (const float *)x_dev, (float *)y_dev, batch, seq, index_pos));
@@ -3075,7 +3232,7 @@ extern "C" int cake_b200_forward_batch_host(cake_b200_ctx *c, cake_b200_block *c
   if (index_pos < 0 || (long long)index_pos + (long long)seq > (long long)kc->cap)
     return fail(CAKE_B200_ESTATE, "index_pos %d + seq %d exceeds cache capacity %d", index_pos, seq, kc->cap);
   CU(cudaSetDevice(c->device));
-  const size_t bytes = (size_t)batch * seq * c->cfg.hidden * (c->cfg.layer_list ? sizeof(float) : c->es);
+  const size_t bytes = (size_t)batch * seq * std::max(1, c->cfg.streams) * c->cfg.hidden * (c->cfg.layer_list ? sizeof(float) : c->es);
   RC(io_reserve(c, bytes));
   memcpy(c->h_pin_x, x_host, bytes);
   CU(cudaMemcpyAsync(c->io_x, c->h_pin_x, bytes, cudaMemcpyHostToDevice, c->stream));
@@ -3126,7 +3283,7 @@ extern "C" int cake_b200_embed(cake_b200_ctx *c, const uint32_t *ids_host, int b
     return DISPATCH_T3(c->cfg.dtype, T_LAMBDA {
       typedef typename decltype(tag_)::type T;
       return launch_pdl(c, embed_f32_kernel<T>, dim3((unsigned)n), dim3(128), 0, (const T *)c->embed, (const uint32_t *)c->d_ids,
-                        (float *)x_dev, (int)n, c->cfg.hidden, c->cfg.vocab, c->cfg.embed_scale);
+                        (float *)x_dev, (int)n, c->cfg.hidden, c->cfg.vocab, c->cfg.embed_scale, std::max(1, c->cfg.streams));
     });
   RC(DISPATCH_T(c->cfg.dtype, T_LAMBDA {
       typedef typename decltype(tag_)::type T;
@@ -3140,6 +3297,7 @@ extern "C" int cake_b200_embed(cake_b200_ctx *c, const uint32_t *ids_host, int b
 extern "C" int cake_b200_head_load_tables(cake_b200_ctx *c, const cake_b200_embed_tables *t) {
   if (!c || !t) return fail(CAKE_B200_EINVAL, "null argument");
   if (!c->cfg.layer_list) return fail(CAKE_B200_EINVAL, "head_load_tables is for models with an fp32 residual stream");
+  if (c->cfg.streams > 0) return fail(CAKE_B200_EINVAL, "head tables are not built for models with several residual streams");
   if ((t->bigram && (t->bigram_rows < 2 || t->mul_prev < 0 || t->mul_cur < 0)) || (t->pos && t->pos_rows < 1)) return fail(CAKE_B200_EINVAL, "bad embedding table sizes");
   CU(cudaSetDevice(c->device));
   const size_t H = c->cfg.hidden;
@@ -3174,7 +3332,7 @@ extern "C" int cake_b200_head_load_tables(cake_b200_ctx *c, const cake_b200_embe
 
 extern "C" int cake_b200_embed_at(cake_b200_ctx *c, cake_b200_cache *kc, const uint32_t *ids_host, int batch, int seq, int index_pos, void *x_dev) {
   if (!c || !kc || !ids_host || !x_dev || !c->embed) return fail(CAKE_B200_EINVAL, "null argument or head not loaded");
-  if (!c->cfg.layer_list) return fail(CAKE_B200_EINVAL, "embed_at is for models with an fp32 residual stream");
+  if (!c->cfg.layer_list || c->cfg.streams > 0) return fail(CAKE_B200_EINVAL, "embed_at is for models with one fp32 residual stream");
   if (batch < 1 || seq < 1 || batch != kc->batch) return fail(CAKE_B200_EINVAL, "embed_at: batch %d (cache batch %d) / seq %d", batch, kc ? kc->batch : 0, seq);
   if (index_pos != kc->embed_len) return fail(CAKE_B200_ESTATE, "embed_at: index_pos %d != the position %d the embedding has reached in this cache", index_pos, kc->embed_len);
   if (c->pos_tab && index_pos + seq > c->pos_rows) return fail(CAKE_B200_ESTATE, "position %d exceeds the %d learned positions", index_pos + seq, c->pos_rows);
@@ -3228,6 +3386,10 @@ static int listed_logits(cake_b200_ctx *c, const void *x_dev, const int *rows_ho
       mx::TanhNorm fn{(const float *)x_dev, rows_host ? c->sp_rows_idx : nullptr, row_mul, row_add, c->ln_f, c->ln_f_b, c->final_alpha, nullptr, nullptr,
                       c->sp_hn, n, (int)H};
       MX(mx::tanh_norm(c->stream, c->cfg.dtype, fn, &c->launches));
+    } else if (c->cfg.streams > 0) {  // the norm of the streams' sum
+      mx::StreamMix sm{(const float *)x_dev, nullptr, nullptr, nullptr, nullptr, nullptr, 0, 0, nullptr, nullptr, 0.f, nullptr, c->ln_f, c->sp_hn, n, (int)H,
+                       c->cfg.streams, c->cfg.rms_eps, rows_host ? c->sp_rows_idx : nullptr, row_mul, row_add};
+      MX(mx::stream_mix(c->stream, c->cfg.dtype, sm, &c->launches));
     } else
     RC(launch_pdl(c, norm_shift_rows_kernel<T>, dim3(n), dim3(256), 0, (const float *)x_dev, (const int *)(rows_host ? c->sp_rows_idx : nullptr),
                   row_mul, row_add, (const T *)c->ln_f,

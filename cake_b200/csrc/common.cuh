@@ -76,6 +76,15 @@ template <typename T> __device__ __forceinline__ float gated_pair(float g, float
   return gate_act<T>(g, act) * u;
 }
 
+// act(z) of a feed-forward without a gate, from the fp32 accumulator: 0 silu, 1 tanh-gelu, 3 relu.  0.5 (1 + tanh t) = sigmoid(2 t);
+// 16-bit D takes the fast exponential and division (its rounding is far coarser)
+template <typename T> __device__ __forceinline__ float plain_act(float z, int act) {
+  if (act == 3) return fmaxf(z, 0.f);
+  const float t = act == 1 ? 1.5957691216057308f * z * (1.0f + 0.044715f * z * z) : z;
+  if (sizeof(T) == 2) return __fdividef(z, 1.0f + __expf(-t));
+  return z / (1.0f + expf(-t));
+}
+
 __device__ __forceinline__ float warp_sum(float v) {
 #pragma unroll
   for (int o = 16; o > 0; o >>= 1) v += __shfl_xor_sync(0xffffffffu, v, o);

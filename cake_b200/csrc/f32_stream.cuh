@@ -6,7 +6,7 @@
 //                            the operands of the matrix products leave in D
 //   gemm_rows_kernel         C = A[M,K] · W[N,K]^T on the CUDA cores, fp32 accumulation, with the epilogues this block needs:
 //                            store in D | act(gate) * up on row-interleaved gate/up | fp32 residual add | soft-capped fp32
-//                            logits.  It serves every shape and D = float (true fp32: one FFMA per product, no TF32); the
+//                            logits | act(C) in D.  It serves every shape and D = float (true fp32: one FFMA per product, no TF32); the
 //                            tcgen05 GEMM (gemm_tc.cuh) takes over for 16-bit D at the shapes its tiles cover.
 //   rows_to_cache_kernel     appends a column range of a row-major activation to a [batch, kv_heads, cap, head_dim] cache
 //
@@ -21,7 +21,7 @@ template <typename T> struct EmbedBits { typedef T type; };
 template <> struct EmbedBits<float> { typedef __nv_bfloat16 type; };  // never taken for float (sizeof test); keeps unpack8 instantiable
 template <typename T>
 __global__ void embed_f32_kernel(const T *__restrict__ E, const uint32_t *__restrict__ ids, float *__restrict__ x, int n_tok,
-                                 int H, int vocab, float scale /* 0 = none */) {
+                                 int H, int vocab, float scale /* 0 = none */, int copies /* rows of x per token, all equal */) {
   pdl_launch_dependents();
   pdl_wait();
   const int t = blockIdx.x;
@@ -29,21 +29,23 @@ __global__ void embed_f32_kernel(const T *__restrict__ E, const uint32_t *__rest
   uint32_t id = ids[t];
   if (id >= (uint32_t)vocab) id = 0;
   const T *src = E + (size_t)id * H;
-  float *dst = x + (size_t)t * H;
+  float *dst = x + (size_t)t * copies * H;
   if (sizeof(T) == 2 && (H & 7) == 0 && scale == 0.f) {  // 16-byte loads, two 16-byte stores per thread and step
     const uint4 *s4 = reinterpret_cast<const uint4 *>(src);
     float4 *d4 = reinterpret_cast<float4 *>(dst);
     for (int i = threadIdx.x; i < H / 8; i += blockDim.x) {
       float f[8];
       unpack8<typename EmbedBits<T>::type>(s4[i], f);
-      d4[2 * i] = make_float4(f[0], f[1], f[2], f[3]);
-      d4[2 * i + 1] = make_float4(f[4], f[5], f[6], f[7]);
+      for (int c = 0; c < copies; c++) {
+        d4[(size_t)c * (H / 4) + 2 * i] = make_float4(f[0], f[1], f[2], f[3]);
+        d4[(size_t)c * (H / 4) + 2 * i + 1] = make_float4(f[4], f[5], f[6], f[7]);
+      }
     }
     return;
   }
   for (int i = threadIdx.x; i < H; i += blockDim.x) {
     const float v = DT<T>::to_f(src[i]);
-    dst[i] = scale == 0.f ? v : v * scale;
+    for (int c = 0; c < copies; c++) dst[(size_t)c * H + i] = scale == 0.f ? v : v * scale;
   }
 }
 
@@ -152,12 +154,12 @@ __global__ void __launch_bounds__(256) norm_shift_rows_kernel(const float *__res
 }
 
 // ---- generic GEMM with the fp32-stream epilogues --------------------------------------------------------------------------
-enum { RE_STORE = 0, RE_GATE_UP = 1, RE_RESIDUAL_F32 = 2, RE_SOFTCAP_F32 = 3 };
+enum { RE_STORE = 0, RE_GATE_UP = 1, RE_RESIDUAL_F32 = 2, RE_SOFTCAP_F32 = 3, RE_ACT = 4 };
 struct RowsGemm {
   const void *A;    // [M, lda] D
   const void *W;    // [N, K] D
   const float *R;   // RE_RESIDUAL_F32: [M, N] fp32
-  void *C;          // RE_STORE: [M, ldc] D;  RE_GATE_UP: [M, ldc] D, N/2 columns written;  else [M, N] fp32
+  void *C;          // RE_STORE / RE_ACT: [M, ldc] D;  RE_GATE_UP: [M, ldc] D, N/2 columns written;  else [M, N] fp32
   int M, N, K, lda, ldc;
   int act;          // RE_GATE_UP: 0 silu, 1 tanh-gelu, 2 clamped (gated_pair; the limit travels in cap)
   float cap;        // RE_SOFTCAP_F32: 0 = none
@@ -212,6 +214,7 @@ __global__ void __launch_bounds__(256) gemm_rows_kernel(const RowsGemm p) {
         const int n = n0 + tx * 4 + j;
         if (n >= p.N) continue;
         if (EPI == RE_STORE) reinterpret_cast<T *>(p.C)[(size_t)m * p.ldc + n] = DT<T>::from_f(p.bias ? acc[i][j] + DT<T>::to_f(reinterpret_cast<const T *>(p.bias)[n]) : acc[i][j]);
+        else if (EPI == RE_ACT) reinterpret_cast<T *>(p.C)[(size_t)m * p.ldc + n] = DT<T>::from_f(plain_act<T>(acc[i][j], p.act));
         else if (EPI == RE_RESIDUAL_F32) reinterpret_cast<float *>(p.C)[(size_t)m * p.N + n] = p.R[(size_t)m * p.N + n] + (p.rs ? p.rs[m] * acc[i][j] : acc[i][j]);
         else reinterpret_cast<float *>(p.C)[(size_t)m * p.N + n] = p.cap > 0.f ? p.cap * tanhf(acc[i][j] / p.cap) : acc[i][j];
       }

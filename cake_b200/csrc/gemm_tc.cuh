@@ -38,14 +38,15 @@ constexpr int TC_SMEM_BYTES = TcCfg<256>::SMEM_BYTES > TcCfg<128>::SMEM_BYTES ? 
 // TCE_RESIDUAL_F32: C (fp32) = residual (fp32) + accumulator, nothing rounded to D — the output projection of a block whose
 // residual stream is fp32 (f32_stream.cuh)
 // TCE_SOFTCAP_F32: C (fp32) = cap * tanh(accumulator / cap) (cap == 0: the accumulator itself) — fp32 logits of such a model
-enum { TCE_PLAIN = 0, TCE_RESIDUAL = 1, TCE_SWIGLU = 2, TCE_RESIDUAL_F32 = 3, TCE_SOFTCAP_F32 = 4 };
+// TCE_ACT: C (D) = act(accumulator), a feed-forward without a gate
+enum { TCE_PLAIN = 0, TCE_RESIDUAL = 1, TCE_SWIGLU = 2, TCE_RESIDUAL_F32 = 3, TCE_SOFTCAP_F32 = 4, TCE_ACT = 5 };
 
 struct TcParams {
   const void *bias;      // [N] D or nullptr (TCE_PLAIN)
   const void *residual;  // [M,N] D (TCE_RESIDUAL)
   void *C;               // [M,N] D  ([M,N/2] for TCE_SWIGLU)
   int M, N, K;
-  int act;  // TCE_SWIGLU: 0 silu, 1 gelu_tanh, 2 the clamped form of gated_pair (its limit travels in cap)
+  int act;  // TCE_ACT: as plain_act; TCE_SWIGLU: 0 silu, 1 gelu_tanh, 2 the clamped form of gated_pair (its limit travels in cap)
   int ldc;  // TCE_SWIGLU / TCE_PLAIN: row stride of C in elements when it is a column range of a wider buffer (0 = N/2 resp. N;
             // a multiple of 8, like the column offset folded into C)
   float cap; // TCE_SOFTCAP_F32; TCE_SWIGLU with act 2: the limit
@@ -327,7 +328,14 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_constant_
             }
 #pragma unroll
             for (int j = 0; j < 16; j++) {
-              float v0 = rnd<T>(__uint_as_float(r[2 * j])), v1 = rnd<T>(__uint_as_float(r[2 * j + 1]));
+              float v0, v1;
+              if (EPI == TCE_ACT) {
+                v0 = plain_act<T>(__uint_as_float(r[2 * j]), p.act);
+                v1 = plain_act<T>(__uint_as_float(r[2 * j + 1]), p.act);
+              } else {
+                v0 = rnd<T>(__uint_as_float(r[2 * j]));
+                v1 = rnd<T>(__uint_as_float(r[2 * j + 1]));
+              }
               if (EPI == TCE_PLAIN && bias) {
                 v0 = rnd<T>(v0 + DT<T>::to_f(bias[n0 + c0 + 2 * j]));
                 v1 = rnd<T>(v1 + DT<T>::to_f(bias[n0 + c0 + 2 * j + 1]));

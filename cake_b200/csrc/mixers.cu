@@ -449,7 +449,7 @@ __global__ void recurrence_kernel(const Recurrence p) {
   extern __shared__ float sm[];
   const int h = blockIdx.x, b = blockIdx.y, dk = p.dk, dv = p.dv;
   const int RS = max(1, (int)blockDim.x / dv);
-  float *St = sm, *qs = St + (size_t)dk * dv, *ks = qs + dk, *vs = ks + dk, *part = vs + dv;
+  float *St = sm, *qs = St + (size_t)dk * dv, *ks = qs + dk, *vs = ks + dk, *part = vs + dv, *av = part + (size_t)RS * dv;
   float *gstate = p.state + ((size_t)b * p.heads + h) * dk * dv;
   for (int i = threadIdx.x; i < dk * dv; i += blockDim.x) St[i] = p.pos0 > 0 ? gstate[i] : 0.f;
   const int gcol = (h / p.group_div) * dk, half = p.rope_dims >> 1;
@@ -482,9 +482,10 @@ __global__ void recurrence_kernel(const Recurrence p) {
         qs[i] = rotated<T>(qr, i, p.rope_dims, cs, sn);
         ks[i] = rotated<T>(kr, i, p.rope_dims, cs, sn) * bsc;
       } else {
-        qs[i] = DT<T>::to_f(qr[i]);
+        qs[i] = DT<T>::to_f(qr[i]) * p.qscale;
         ks[i] = DT<T>::to_f(kr[i]) * bsc;
       }
+      if (p.a_chan) av[i] = p.a_chan[(m * p.heads + h) * dk + i];
     }
     for (int i = threadIdx.x; i < dv; i += blockDim.x) vs[i] = DT<T>::to_f(vr[i]);
     __syncthreads();
@@ -493,7 +494,7 @@ __global__ void recurrence_kernel(const Recurrence p) {
         const float v = vs[jj];
         float acc = 0.f;
         for (int i = s; i < dk; i += RS) {
-          const float sn_ = fmaf(a, St[(size_t)i * dv + jj], ks[i] * v);
+          const float sn_ = fmaf(p.a_chan ? av[i] : a, St[(size_t)i * dv + jj], ks[i] * v);
           St[(size_t)i * dv + jj] = sn_;
           acc = fmaf(sn_, qs[i], acc);
         }
@@ -662,7 +663,12 @@ template <typename T, int R> static cudaError_t launch_recurrence_cols(cudaStrea
 
 int recurrence(cudaStream_t st, int dtype, const Recurrence &p, uint64_t *launches) {
   if (p.dv > 1024 || p.dk < 1) return (int)cudaErrorInvalidValue;
-  if (p.dk % RC_RS == 0 && p.dv % RC_CB == 0) {
+  if (p.a_chan) {
+    if (p.dt || p.a_tok || p.skip || p.cos_t || p.group_div != 1) return (int)cudaErrorInvalidValue;
+    const int e = recurrence_channels(st, dtype, p);
+    if (e == (int)cudaSuccess) MX_DONE(1);
+    if (e != (int)cudaErrorNotSupported) return e;
+  } else if (p.dk % RC_RS == 0 && p.dv % RC_CB == 0) {
     cudaError_t e = cudaErrorNotSupported;
     MX_DISPATCH(dtype, {
       switch (p.dk / RC_RS) {
@@ -681,7 +687,7 @@ int recurrence(cudaStream_t st, int dtype, const Recurrence &p, uint64_t *launch
   }
   const int threads = p.dv <= 256 ? 256 : (p.dv + 31) / 32 * 32;
   const int RS = threads / p.dv > 0 ? threads / p.dv : 1;
-  const size_t smem = ((size_t)p.dk * p.dv + 2 * p.dk + p.dv + (size_t)RS * p.dv) * sizeof(float);
+  const size_t smem = ((size_t)p.dk * p.dv + (p.a_chan ? 3 : 2) * (size_t)p.dk + p.dv + (size_t)RS * p.dv) * sizeof(float);
   if (smem > 227 * 1024) return (int)cudaErrorInvalidValue;
   MX_DISPATCH(dtype, {
     static int attr_dev = -1;
@@ -922,7 +928,8 @@ __global__ void __launch_bounds__(128) moe_router_kernel(const MoePlan p) {
   float sum = 0.f, sc[NS], ch[NS];
 #pragma unroll
   for (int sI = 0; sI < NS; sI++) {
-    sc[sI] = lane + 32 * sI < E ? expf(z[sI] - mx) : 0.f;
+    if (p.sigmoid_scores) sc[sI] = 1.0f / (1.0f + expf(-z[sI]));   // lanes past the last expert: z = -inf, a score of zero
+    else sc[sI] = lane + 32 * sI < E ? expf(z[sI] - mx) : 0.f;
     sum += sc[sI];
   }
   sum = warp_sum(sum);
@@ -933,7 +940,7 @@ __global__ void __launch_bounds__(128) moe_router_kernel(const MoePlan p) {
       ch[sI] = z[sI];
       continue;
     }
-    sc[sI] = sc[sI] / sum;
+    if (!p.sigmoid_scores) sc[sI] = sc[sI] / sum;
     ch[sI] = e < E ? sc[sI] + (corr ? DT<T>::to_f(corr[e]) : 0.f) : -INFINITY;
   }
   if (p.groups > 1) {  // lane g keeps the best score of group g (g = lane + 32 sI); the best groups_keep groups stay open
@@ -1102,12 +1109,27 @@ int moe_route(cudaStream_t st, int dtype, const MoePlan &p, uint64_t *launches) 
 }
 
 template <typename T>
-__global__ void __launch_bounds__(128) moe_gather_kernel(const T *__restrict__ h, const int *__restrict__ perm, T *__restrict__ sorted, int W, int top) {
+__global__ void __launch_bounds__(128) moe_gather_kernel(const T *__restrict__ h, const int *__restrict__ perm, T *__restrict__ sorted, int W, int top,
+                                                         const float *__restrict__ wts) {
   const size_t r = blockIdx.x;
   const int e = perm[r];
   T *dst = sorted + r * W;
   const T *src = e >= 0 ? h + (size_t)(e / top) * W : nullptr;
   constexpr int VE = 16 / (int)sizeof(T);
+  if (wts && src) {
+    const float w = wts[e];
+    if (W % 4 == 0) {
+      for (int i = threadIdx.x; i < W / 4; i += blockDim.x) {
+        float v[4];
+        load4<T>(src + 4 * i, v);
+        v[0] *= w; v[1] *= w; v[2] *= w; v[3] *= w;
+        store4<T>(dst + 4 * i, v);
+      }
+      return;
+    }
+    for (int i = threadIdx.x; i < W; i += blockDim.x) dst[i] = DT<T>::from_f(w * DT<T>::to_f(src[i]));
+    return;
+  }
   if (W % VE == 0) {
     for (int i = threadIdx.x; i < W / VE; i += blockDim.x)
       reinterpret_cast<uint4 *>(dst)[i] = src ? reinterpret_cast<const uint4 *>(src)[i] : make_uint4(0, 0, 0, 0);
@@ -1115,8 +1137,8 @@ __global__ void __launch_bounds__(128) moe_gather_kernel(const T *__restrict__ h
   }
   for (int i = threadIdx.x; i < W; i += blockDim.x) dst[i] = src ? src[i] : DT<T>::from_f(0.f);
 }
-int moe_gather(cudaStream_t st, int dtype, const void *h, const int *perm, void *sorted, int rows, int W, int top, uint64_t *launches) {
-  MX_DISPATCH(dtype, (moe_gather_kernel<T><<<rows, 128, 0, st>>>(reinterpret_cast<const T *>(h), perm, reinterpret_cast<T *>(sorted), W, top)));
+int moe_gather(cudaStream_t st, int dtype, const void *h, const int *perm, void *sorted, int rows, int W, int top, uint64_t *launches, const float *wts) {
+  MX_DISPATCH(dtype, (moe_gather_kernel<T><<<rows, 128, 0, st>>>(reinterpret_cast<const T *>(h), perm, reinterpret_cast<T *>(sorted), W, top, wts)));
   MX_DONE(1);
 }
 
@@ -1151,6 +1173,7 @@ __global__ void __launch_bounds__(256) moe_expert_kernel(const MoeExperts p) {
       if (src[r] >= 0 && k0 + c < K) {
         const size_t arow = PHASE == 0 ? (size_t)(src[r] / p.top) : (size_t)(row0 + r);
         a = DT<T>::to_f(A[arow * K + k0 + c]);
+        if (PHASE == 0 && p.in_wts) a *= p.in_wts[src[r]];
       }
       As[c][r] = a;
       const bool ok = n0 + r < N && k0 + c < K;
@@ -1222,7 +1245,7 @@ __global__ void __launch_bounds__(256) moe_combine_kernel(const MoeCombine p) {
       float4 s = x4 ? x4[i] : make_float4(0.f, 0.f, 0.f, 0.f);
       for (int k = 0; k < p.top; k++) {
         const size_t pr = (size_t)m * p.top + k;
-        const float w = p.wts[pr];
+        const float w = p.wts ? p.wts[pr] : 1.f;
         if (p.ids[pr] < p.experts) {
           const float4 y = reinterpret_cast<const float4 *>(p.y + (size_t)p.pos_of[pr] * p.W)[i];
           s.x = fmaf(w, y.x, s.x); s.y = fmaf(w, y.y, s.y); s.z = fmaf(w, y.z, s.z); s.w = fmaf(w, y.w, s.w);
@@ -1240,7 +1263,7 @@ __global__ void __launch_bounds__(256) moe_combine_kernel(const MoeCombine p) {
     for (int k = 0; k < p.top; k++) {
       const size_t pr = (size_t)m * p.top + k;
       const int e = p.ids[pr];
-      s = fmaf(p.wts[pr], e < p.experts ? p.y[(size_t)p.pos_of[pr] * p.W + i] : DT<T>::to_f(h[i]), s);
+      s = fmaf(p.wts ? p.wts[pr] : 1.f, e < p.experts ? p.y[(size_t)p.pos_of[pr] * p.W + i] : DT<T>::to_f(h[i]), s);
     }
     p.x_out[(size_t)m * p.W + i] = (p.x ? p.x[(size_t)m * p.W + i] : 0.f) + s;
   }
@@ -1438,7 +1461,7 @@ template <typename T> __device__ __forceinline__ float4 merge_load(const StreamM
   for (int k = 0; k < p.top; k++) {
     const size_t pr = (size_t)m * p.top + k;
     if (p.ids[pr] >= p.experts) continue;
-    const float w = p.wts[pr];
+    const float w = p.wts ? p.wts[pr] : 1.f;
     const float4 y = reinterpret_cast<const float4 *>(p.y + (size_t)p.pos_of[pr] * p.n)[i4];
     s.x = fmaf(w, y.x, s.x); s.y = fmaf(w, y.y, s.y); s.z = fmaf(w, y.z, s.z); s.w = fmaf(w, y.w, s.w);
   }
@@ -1494,7 +1517,7 @@ __global__ void __launch_bounds__(256) stream_merge_any_kernel(const StreamMerge
     else
       for (int k = 0; k < p.top; k++) {
         const size_t pr = (size_t)m * p.top + k;
-        if (p.ids[pr] < p.experts) v = fmaf(p.wts[pr], p.y[(size_t)p.pos_of[pr] * p.n + i], v);
+        if (p.ids[pr] < p.experts) v = fmaf(p.wts ? p.wts[pr] : 1.f, p.y[(size_t)p.pos_of[pr] * p.n + i], v);
       }
     ys[i] = v;
     ss = fmaf(v, v, ss);
@@ -1511,7 +1534,7 @@ __global__ void __launch_bounds__(256) stream_merge_any_kernel(const StreamMerge
   }
 }
 int stream_merge(cudaStream_t st, int dtype, const StreamMerge &p, uint64_t *launches) {
-  if (p.M < 1 || p.n < 1 || !p.x || !p.x_out || (!p.a && (!p.y || !p.wts || !p.ids || !p.pos_of || p.top < 1))) return (int)cudaErrorInvalidValue;
+  if (p.M < 1 || p.n < 1 || !p.x || !p.x_out || (!p.a && (!p.y || !p.ids || !p.pos_of || p.top < 1))) return (int)cudaErrorInvalidValue;
   const bool vec = p.n % 4 == 0 && p.n <= 8192 && (((uintptr_t)p.a | (uintptr_t)p.y | (uintptr_t)p.x | (uintptr_t)p.x_out | (uintptr_t)p.xd) & 15) == 0;
   const size_t smem = (size_t)p.n * sizeof(float);
   if (!vec && smem > 200 * 1024) return (int)cudaErrorInvalidValue;

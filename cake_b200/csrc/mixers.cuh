@@ -97,8 +97,26 @@ struct Recurrence {
   int B, S, heads, dk, dv, pos0;
   // per-token factors computed elsewhere: a_t = a_tok[m, h], b_t = b_tok[m, h] (fp32 [M, heads]); they override decay / dt
   const float *a_tok = nullptr, *b_tok = nullptr;
+  // a decay per key channel: S_t = diag(a_chan[m, h * dk ..]) S_{t-1} + kscale k_t v_t^T (fp32 [M, heads * dk]; no rotation, group_div 1,
+  // no dt / a_tok / skip); q is multiplied by qscale
+  const float *a_chan = nullptr;
+  float qscale = 1.f;
 };
 int recurrence(cudaStream_t, int dtype, const Recurrence &, uint64_t *launches);
+// the register-tiled form with a decay per key channel; cudaErrorNotSupported for shapes it does not cover (recurrence() then
+// takes the kernel with the state in shared memory)
+int recurrence_channels(cudaStream_t, int dtype, const Recurrence &);
+
+// ---- decays per key channel from a low-rank product: a = sigmoid(W u + bias)^(1 / tau) --------------------------------------
+struct ChannelDecay {
+  const void *u;         // [M, ld] D, rank entries
+  int ld, rank;
+  const void *w, *bias;  // [channels, rank], [channels] D
+  float *a;              // [M, channels] fp32
+  int M, channels;
+  float tau;
+};
+int channel_decay(cudaStream_t, int dtype, const ChannelDecay &, uint64_t *launches);
 
 // ---- short causal convolution per channel + silu -----------------------------------------------------------------------
 struct ShortConv {
@@ -155,11 +173,14 @@ struct MoePlan {
   // groups > 1: the experts form that many equal groups of neighbours, only those of the groups_keep groups with the largest best
   // score s may be chosen; plain_weights: the weights are the scores s (times scale), not renormalised.  correction may be nullptr
   int groups = 0, groups_keep = 0, plain_weights = 0;
+  int sigmoid_scores = 0;  // 1: s = sigmoid(z) instead of the softmax
 };
 int moe_route(cudaStream_t, int dtype, const MoePlan &, uint64_t *launches);
 
 // sorted[r] = h[perm[r] / top] (zeros for padding rows): the operand of a grouped product on the tensor cores
-int moe_gather(cudaStream_t, int dtype, const void *h, const int *perm, void *sorted, int rows, int W, int top, uint64_t *launches);
+// (wts [M, top] != nullptr: times the pair's weight, rounded to D once)
+int moe_gather(cudaStream_t, int dtype, const void *h, const int *perm, void *sorted, int rows, int W, int top, uint64_t *launches,
+               const float *wts = nullptr);
 
 // CUDA-core experts for every shape and D = float: act = f(Wg h) * (Wu h), then y[sorted row] = Wd act
 struct MoeExperts {
@@ -172,6 +193,7 @@ struct MoeExperts {
   const int *perm, *tile_expert;
   int tile, max_tiles;
   float limit = 0.f;     // act_kind 2 (the clamped form): its limit
+  const float *in_wts = nullptr;  // [M, top]: a pair's expert reads its weight times h
 };
 int moe_experts(cudaStream_t, int dtype, const MoeExperts &, uint64_t *launches);
 
@@ -181,7 +203,7 @@ struct MoeCombine {
   const float *x;
   float *x_out;
   const void *h;         // [M, W] D
-  const float *y, *wts;
+  const float *y, *wts;  // wts nullptr: every weight is one
   const int *ids, *pos_of;
   int M, W, top, experts;
 };
@@ -229,7 +251,7 @@ int branch_merge(cudaStream_t, int dtype, const BranchMerge &, uint64_t *launche
 //   x_out = x + (post ? rms(y) * post : y);   xd (nullable) = x_out rounded to D: the next sublayer's operand
 struct StreamMerge {
   const float *a;        // [M, n] fp32, or nullptr with the routed sum below
-  const float *y, *wts;  // [sorted rows, n], [M, top]
+  const float *y, *wts;  // [sorted rows, n], [M, top] (nullptr: every weight is one)
   const int *ids, *pos_of;  // [M, top]; slots whose id is not below `experts` add nothing
   int top, experts;
   const void *post;      // [n] D or nullptr
@@ -240,6 +262,32 @@ struct StreamMerge {
   float eps;
 };
 int stream_merge(cudaStream_t, int dtype, const StreamMerge &, uint64_t *launches);
+
+// ---- several residual streams per token ---------------------------------------------------------------------------------------
+// One pass over a token's streams X_s (rows of [streams, n] fp32) between two sublayers:
+//   y = (a ? a : 0) + (routed ? sum over slots of y_sorted[pos_of] : 0)                       (the sublayer's output)
+//   X_t <- sum_s mix[s, t] X_s + mult out[t] y                                              (mix == nullptr: the streams stay as they are)
+//   u = sum_s in[s] X_s (in == nullptr: the plain sum);  h = u / rms(u) * w                  (h == nullptr: nothing is read out)
+// With rows / row_mul the read-out alone is made for chosen rows (the head): source row = rows ? rows[m] : m * row_mul + row_add.
+struct StreamMix {
+  const float *x;        // [*, streams, n]
+  float *x_out;          // may alias x
+  const float *a;        // [M, n] or nullptr
+  const float *y;        // sorted expert rows or nullptr
+  const int *ids, *pos_of;  // [M, top]; slots whose id is not below `experts` add nothing
+  int top, experts;
+  const void *mix, *out; // [streams, streams], [streams] D
+  float mult;
+  const void *in;        // [streams] D or nullptr
+  const void *w;         // [n] D
+  void *h;               // [M, n] D or nullptr
+  int M, n, streams;
+  float eps;
+  const int *rows = nullptr;
+  int row_mul = 1, row_add = 0;
+};
+constexpr int MAX_STREAMS = 16;
+int stream_mix(cudaStream_t, int dtype, const StreamMix &, uint64_t *launches);
 
 // ---- gated delta rule -----------------------------------------------------------------------------------------------------
 // Prep: q and k of every key head become unit vectors (x / sqrt(sum x^2 + 1e-6); q also times qscale) in fp32, and per head
@@ -400,6 +448,8 @@ struct QkPrep {
   int interleaved = 0;   // 1: pairs (2i, 2i + 1) instead of (i, i + rope_dims / 2)
   const void *q_w = nullptr, *k_w = nullptr;  // [dim] D: every head is x / rms(x) * gain IN FRONT OF the rotation (instead of unit_norm)
   int v_unit = 0;        // 1: every value head is divided by its root mean square
+  int wide_norm = 0;     // 1: q_w [heads * dim], k_w [kv_heads * dim]: one RMS norm over the whole projection, in front of the rotation
+                         // kv_heads == 0: queries alone
 };
 int qk_prep(cudaStream_t, int dtype, const QkPrep &, uint64_t *launches);
 

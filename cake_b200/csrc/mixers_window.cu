@@ -286,6 +286,108 @@ __global__ void __launch_bounds__(256) qk_prep_vec_kernel(const QkPrep p) {
         *reinterpret_cast<const uint4 *>(row + p.v_col + i);
   }
 }
+// One norm over the whole projection of a row (q, and k on its own) in front of the rotation: a CTA per row.
+__device__ __forceinline__ void qk_sums(float &a, float &b, float *red /* [64] */) {
+  a = warp_sum(a);
+  b = warp_sum(b);
+  const int w = threadIdx.x >> 5, nw = blockDim.x >> 5;
+  if ((threadIdx.x & 31) == 0) { red[w] = a; red[32 + w] = b; }
+  __syncthreads();
+  a = b = 0.f;
+  for (int i = 0; i < nw; i++) { a += red[i]; b += red[32 + i]; }
+}
+template <typename T>
+__global__ void __launch_bounds__(256) qk_prep_wide_kernel(const QkPrep p) {
+  __shared__ float red[64];
+  const int m = blockIdx.x, b = m / p.S, t = m % p.S, pos = p.pos0 + t, sq = p.heads * p.dim, sk = p.kv_heads * p.dim;
+  const T *row = reinterpret_cast<const T *>(p.proj) + (size_t)m * p.ld;
+  const int dims = p.cos_t ? p.rope_dims : 0, half = dims >> 1;
+  const float *cs = p.cos_t ? p.cos_t + (size_t)pos * half : nullptr, *sn = p.sin_t ? p.sin_t + (size_t)pos * half : nullptr;
+  float ssq = 0.f, ssk = 0.f;
+  for (int i = threadIdx.x; i < sq; i += blockDim.x) { const float v = DT<T>::to_f(row[p.q_col + i]); ssq = fmaf(v, v, ssq); }
+  for (int i = threadIdx.x; i < sk; i += blockDim.x) { const float v = DT<T>::to_f(row[p.k_col + i]); ssk = fmaf(v, v, ssk); }
+  qk_sums(ssq, ssk, red);
+  const float invq = 1.0f / sqrtf(ssq / (float)sq + p.eps), invk = sk ? 1.0f / sqrtf(ssk / (float)sk + p.eps) : 0.f;
+  for (int i = threadIdx.x; i < sq + sk; i += blockDim.x) {
+    const bool is_q = i < sq;
+    const int hv = (is_q ? i : i - sq) / p.dim, e = (is_q ? i : i - sq) % p.dim;
+    const T *v = row + (is_q ? p.q_col : p.k_col) + (size_t)hv * p.dim, *w = reinterpret_cast<const T *>(is_q ? p.q_w : p.k_w) + (size_t)hv * p.dim;
+    T *o = is_q ? reinterpret_cast<T *>(p.q_out) + ((size_t)m * p.heads + hv) * p.dim
+                : reinterpret_cast<T *>(p.kc) + (((size_t)b * p.kv_heads + hv) * p.cap + pos) * p.dim;
+    o[e] = DT<T>::from_f(rotated_entry<T>(v, e, dims, cs, sn, w, p.interleaved != 0) * (is_q ? invq : invk));
+  }
+  for (int i = threadIdx.x; i < p.kv_heads * p.vdim; i += blockDim.x) {
+    const int g = i / p.vdim, e = i % p.vdim;
+    reinterpret_cast<T *>(p.vc)[(((size_t)b * p.kv_heads + g) * p.cap + pos) * p.vdim + e] = row[p.v_col + i];
+  }
+}
+// The same in 16-byte pieces for 16-bit D and adjacent pairs: thread i owns the pieces i, i + 256, ... of q and then k (NP of them, in
+// registers between the sums and the store); a piece lies inside one head.
+template <typename T, int NP>
+__global__ void __launch_bounds__(256) qk_prep_wide_vec_kernel(const QkPrep p) {
+  __shared__ float red[64];
+  const int m = blockIdx.x, b = m / p.S, t = m % p.S, pos = p.pos0 + t, sq = p.heads * p.dim, sk = p.kv_heads * p.dim;
+  const T *row = reinterpret_cast<const T *>(p.proj) + (size_t)m * p.ld;
+  const int dims = p.cos_t ? p.rope_dims : 0, half = dims >> 1, n8 = (sq + sk) / 8;
+  const float *cs = p.cos_t ? p.cos_t + (size_t)pos * half : nullptr, *sn = p.sin_t ? p.sin_t + (size_t)pos * half : nullptr;
+  uint4 raw[NP];
+  float ssq = 0.f, ssk = 0.f;
+#pragma unroll
+  for (int u = 0; u < NP; u++) {
+    const int i = 8 * (threadIdx.x + 256 * u);
+    raw[u] = make_uint4(0, 0, 0, 0);
+    if (i < 8 * n8) raw[u] = *reinterpret_cast<const uint4 *>(row + (i < sq ? p.q_col + i : p.k_col + i - sq));
+    float f[8], s = 0.f;
+    unpack8<T>(raw[u], f);
+#pragma unroll
+    for (int e = 0; e < 8; e++) s = fmaf(f[e], f[e], s);
+    if (i < sq) ssq += s;
+    else ssk += s;
+  }
+  const int vrow = p.kv_heads * p.vdim;
+  for (int i = threadIdx.x * 8; i < vrow; i += blockDim.x * 8) {
+    const int g = i / p.vdim, e = i % p.vdim;
+    *reinterpret_cast<uint4 *>(reinterpret_cast<T *>(p.vc) + (((size_t)b * p.kv_heads + g) * p.cap + pos) * p.vdim + e) =
+        *reinterpret_cast<const uint4 *>(row + p.v_col + i);
+  }
+  qk_sums(ssq, ssk, red);
+  const float invq = 1.0f / sqrtf(ssq / (float)sq + p.eps), invk = sk ? 1.0f / sqrtf(ssk / (float)sk + p.eps) : 0.f;
+#pragma unroll
+  for (int u = 0; u < NP; u++) {
+    const int i = 8 * (threadIdx.x + 256 * u);
+    if (i >= 8 * n8) continue;
+    const bool is_q = i < sq;
+    const int j = is_q ? i : i - sq, hv = j / p.dim, e0 = j % p.dim;
+    const float inv = is_q ? invq : invk;
+    float f[8], w[8];
+    unpack8<T>(raw[u], f);
+    unpack8<T>(*reinterpret_cast<const uint4 *>(reinterpret_cast<const T *>(is_q ? p.q_w : p.k_w) + j), w);
+    uint32_t o[4];
+#pragma unroll
+    for (int e = 0; e < 4; e++) {
+      const float x = f[2 * e] * w[2 * e] * inv, y = f[2 * e + 1] * w[2 * e + 1] * inv;
+      float c = 1.f, s = 0.f;
+      if (e0 + 2 * e < dims) { c = cs[(e0 >> 1) + e]; s = sn[(e0 >> 1) + e]; }
+      o[e] = pack2x<T>(x * c - y * s, y * c + x * s);
+    }
+    T *dst = is_q ? reinterpret_cast<T *>(p.q_out) + (size_t)m * sq + j
+                  : reinterpret_cast<T *>(p.kc) + (((size_t)b * p.kv_heads + hv) * p.cap + pos) * p.dim + e0;
+    *reinterpret_cast<uint4 *>(dst) = make_uint4(o[0], o[1], o[2], o[3]);
+  }
+}
+template <typename T> static bool qk_prep_wide_vec(cudaStream_t st, const QkPrep &p) {
+  const int n8 = (p.heads + p.kv_heads) * p.dim / 8;
+  const bool ok = p.dim % 8 == 0 && p.vdim % 8 == 0 && p.ld % 8 == 0 && p.q_col % 8 == 0 && p.k_col % 8 == 0 && p.v_col % 8 == 0 && n8 <= 256 * 8 &&
+                  (p.interleaved || !p.cos_t) &&
+                  (((uintptr_t)p.proj | (uintptr_t)p.q_out | (uintptr_t)p.kc | (uintptr_t)p.vc | (uintptr_t)p.q_w | (uintptr_t)p.k_w) & 15) == 0;
+  if (!ok) return false;
+  if (n8 <= 256) qk_prep_wide_vec_kernel<T, 1><<<p.B * p.S, 256, 0, st>>>(p);
+  else if (n8 <= 512) qk_prep_wide_vec_kernel<T, 2><<<p.B * p.S, 256, 0, st>>>(p);
+  else if (n8 <= 1024) qk_prep_wide_vec_kernel<T, 4><<<p.B * p.S, 256, 0, st>>>(p);
+  else qk_prep_wide_vec_kernel<T, 8><<<p.B * p.S, 256, 0, st>>>(p);
+  return true;
+}
+template <> bool qk_prep_wide_vec<float>(cudaStream_t, const QkPrep &) { return false; }
 template <typename T> static bool qk_prep_vec(cudaStream_t st, const QkPrep &p) {
   const int E = p.dim / 32, half = p.cos_t ? p.rope_dims / 2 : 0;
   const bool ok = p.dim % 32 == 0 && (E == 2 || E == 4 || E == 8) && (p.interleaved ? 2 * half : half) % E == 0 && p.vdim % 8 == 0 && p.ld % 8 == 0 && p.q_col % 8 == 0 &&
@@ -302,8 +404,16 @@ template <typename T> static bool qk_prep_vec(cudaStream_t st, const QkPrep &p) 
 }
 template <> bool qk_prep_vec<float>(cudaStream_t, const QkPrep &) { return false; }
 int qk_prep(cudaStream_t st, int dtype, const QkPrep &p, uint64_t *launches) {
-  if (p.B < 1 || p.S < 1 || p.heads < 1 || p.kv_heads < 1 || !p.q_w != !p.k_w || (p.cos_t && (p.rope_dims & 1 || p.rope_dims > p.dim))) return (int)cudaErrorInvalidValue;
+  if (p.B < 1 || p.S < 1 || p.heads < 1 || p.kv_heads < 0 || (p.kv_heads > 0 && (!p.q_w != !p.k_w || !p.kc || !p.vc)) ||
+      (p.wide_norm && (!p.q_w || p.unit_norm || p.v_unit)) || (p.cos_t && (p.rope_dims & 1 || p.rope_dims > p.dim)))
+    return (int)cudaErrorInvalidValue;
   bool done = false;
+  if (p.wide_norm) {
+    MX_DISPATCH(dtype, (done = qk_prep_wide_vec<T>(st, p)));
+    if (done) MX_DONE(1);
+    MX_DISPATCH(dtype, (qk_prep_wide_kernel<T><<<p.B * p.S, 256, 0, st>>>(p)));
+    MX_DONE(1);
+  }
   MX_DISPATCH(dtype, (done = qk_prep_vec<T>(st, p)));
   if (done) MX_DONE(1);
   MX_DISPATCH(dtype, (qk_prep_kernel<T><<<p.B * p.S, (p.heads + p.kv_heads) > 4 ? 256 : 128, 0, st>>>(p)));

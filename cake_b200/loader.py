@@ -491,6 +491,55 @@ def mafosun_block_tensors(vb, cfg: Config, index: int):
     return main, side
 
 
+def lilenex_block_tensors(vb, cfg: Config, index: int) -> Dict[str, object]:
+    """The tensors of layer ``index`` of a Lilenex checkpoint by the field names of ``cake_b200_mixer_tensors``, each checked against the
+    shape its MixerSpec declares.  Names under ``l<i>.``: ``norm1``, ``norm2``, ``hc1.{in,out,mix}``, ``hc2.*`` and ``mix.*``: an attention
+    layer has ``q, q.norm, k, k.norm, v, o`` (with shared keys and values only ``q, q.norm, o``); a gated linear layer ``q, k, v, g, o, norm,
+    a1, a2, a2.b`` (the rows of ``a1`` set the spec's ``decay_rank``); ``mlp.{up,down}`` (dense) or ``mlp.{router, e<j>.*, shared.*}``."""
+    sp, H, name = cfg.layers[index], cfg.hidden_size, cfg.layer_name(index)
+
+    def get(short, shape):
+        t = vb.get(f"{name}.{short}")
+        if t is None:
+            raise KeyError(f"tensor {name}.{short} not found")
+        if tuple(t.shape) != tuple(shape):
+            raise ValueError(f"shape mismatch for {name}.{short}, expected: {list(shape)}, got: {list(t.shape)}")
+        return t
+
+    sq = sp.heads * sp.dim
+    out: Dict[str, object] = dict(norm1=get("norm1", (H,)), q=get("mix.q", (sq, H)), o=get("mix.o", (H, sp.inner)))
+    if sp.type == "sink_attention":
+        out["q_norm"] = get("mix.q.norm", (sq,))
+        if not sp.kv_back:
+            out.update(k=get("mix.k", (sp.n_kv * sp.dim, H)), v=get("mix.v", (sp.n_kv * sp.vdim, H)), k_norm=get("mix.k.norm", (sp.n_kv * sp.dim,)))
+    else:
+        a1 = vb.get(f"{name}.mix.a1")
+        if a1 is not None and a1.dim() == 2:
+            sp.decay_rank = int(a1.shape[0])
+        out.update(k=get("mix.k", (sq, H)), v=get("mix.v", (sp.inner, H)), g=get("mix.g", (sp.inner, H)), norm=get("mix.norm", (sp.vdim,)),
+                   a1=get("mix.a1", (sp.decay_rank, H)), a2=get("mix.a2", (sq, sp.decay_rank)), a2_b=get("mix.a2.b", (sq,)))
+    mo = sp.moe
+    if sp.dense_ff:
+        out.update(ff_up=get("mlp.up", (sp.dense_ff, H)), ff_down=get("mlp.down", (H, sp.dense_ff)))
+    elif mo is not None:
+        out.update(router=get("mlp.router", (mo.experts, H)), e_gate=[get(f"mlp.e{j}.gate", (mo.ff, H)) for j in range(mo.experts)],
+                   e_up=[get(f"mlp.e{j}.up", (mo.ff, H)) for j in range(mo.experts)],
+                   e_down=[get(f"mlp.e{j}.down", (H, mo.ff)) for j in range(mo.experts)])
+        if mo.shared_ff:
+            out.update(s_gate=get("mlp.shared.gate", (mo.shared_ff, H)), s_up=get("mlp.shared.up", (mo.shared_ff, H)),
+                       s_down=get("mlp.shared.down", (H, mo.shared_ff)))
+    n = sp.streams
+    for q in (1, 2) if sp.dense_ff or mo is not None else (1,):
+        if q == 2:
+            out["norm2"] = get("norm2", (H,))
+        for short, shape in (("in", (n,)), ("out", (n,)), ("mix", (n, n))):
+            if n == 1 and vb.get(f"{name}.hc{q}.{short}") is None:   # one stream without coefficients: the plain residual sum
+                out[f"hc{q}_{short}"] = torch.ones(shape)
+            else:
+                out[f"hc{q}_{short}"] = get(f"hc{q}.{short}", shape)
+    return out
+
+
 def detect_model_prefix(index_path: str, configured: str) -> str:
     """cake/mod.rs:335-357: the text before the first ``.layers.0.`` key of the index wins over the configured prefix."""
     if not os.path.exists(index_path):

@@ -327,11 +327,12 @@ def _mixer_struct(sp, views, ctx, keep):
                       CRotarySpec(r.dims, r.base, r.factor, r.fast, r.slow, r.original, int(r.interleaved), *(r.stretch or (0.0, 0.0, 0.0, 0.0))),
                       decay if sp.decay else None, sp.state, sp.groups, sp.conv, sp.norm_groups,
                       CMoeSpec(mo.experts, mo.identity, mo.top, mo.scale, mo.ff, mo.shared_ff, mo.act, mo.limit, mo.shared_limit, int(mo.logit_bias),
-                               mo.groups, mo.groups_keep, int(mo.plain_weights))
+                               mo.groups, mo.groups_keep, int(mo.plain_weights), int(mo.sigmoid_scores), int(mo.weigh_input))
                       if mo else CMoeSpec(),
                       sp.kv_heads, sp.bias_rows, sp.bias_max, sp.gate_cap, sp.norm_offset, sp.canon_taps, sp.dense_ff, sp.dense_act,
                       sp.dense_limit, None, sp.window, sp.keep_first, int(sp.qk_unit), sp.q_rank, sp.norm_kind, (ctypes.c_float * 4)(*sp.norm_alpha),
-                      sp.side_dim, sp.side_col, sp.pool, sp.chunk, sp.softcap, int(sp.sink_zero), int(sp.qk_norm), int(sp.v_unit), sp.branch_scale)
+                      sp.side_dim, sp.side_col, sp.pool, sp.chunk, sp.softcap, int(sp.sink_zero), 2 if sp.qk_norm_wide else int(sp.qk_norm), int(sp.v_unit),
+                      sp.branch_scale, sp.kv_back, sp.decay_rank, sp.decay_tau, sp.streams, sp.residual_mult)
     return spec, CMixerTensors(**args)
 
 
@@ -400,9 +401,27 @@ class OutputNormBlock(MixerBlock):
         return cls(name, h, ctx)
 
 
+class StreamsBlock(MixerBlock):
+    """A layer of a Lilenex model: a mixer-list block (``cake_b200_block_load_mixer``) with several residual streams, whose mixer is
+    windowed attention (its keys and values possibly another layer's) or gated linear attention; a dense feed-forward without a gate or
+    a routed one with sigmoid scores on the experts' inputs.  Activations between blocks are [batch, seq, streams * hidden] fp32."""
+
+    @classmethod
+    def load(cls, name: str, ctx: Context) -> "StreamsBlock":
+        from .loader import lilenex_block_tensors
+        cfg = ctx.config
+        index = [cfg.layer_name(i) for i in range(len(cfg.layers))].index(name)
+        views = lilenex_block_tensors(ctx.var_builder, cfg, index)   # also fills the spec's decay_rank
+        keep = []
+        spec, tens = _mixer_struct(cfg.layers[index], views, ctx, keep)
+        h = c_void_p()
+        check(lib().cake_b200_block_load_mixer(ctx.h, index, byref(spec), byref(tens), byref(h)))
+        return cls(name, h, ctx)
+
+
 # Config.block_kind -> the Forwarder that loads and runs its layers
 BLOCK_CLASSES = {"nigenex": ListedBlock, "setodra": MixerBlock, "nuvarax": SandwichBlock, "netolorn": SquashBlock,
-                 "mafosun": OutputNormBlock}
+                 "mafosun": OutputNormBlock, "lilenex": StreamsBlock}
 
 
 @dataclass
@@ -502,7 +521,7 @@ class TextModelBase:
         ids = np.ascontiguousarray(ids, dtype=np.uint32)
         b, s = ids.shape
         ctx = self.ctx
-        x = ctx.empty(b, s, ctx.config.hidden_size, dtype=ctx.stream_dtype)
+        x = ctx.empty(b, s, ctx.config.stream_width, dtype=ctx.stream_dtype)
         if getattr(self, "embed_at", False):   # the cache supplies the previous token of every row and checks the position
             check(lib().cake_b200_embed_at(ctx.h, ctx.cache.h, ids.ctypes.data_as(ctypes.POINTER(c_uint32)), b, s, idx, ptr(x)))
         else:

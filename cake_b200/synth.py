@@ -376,3 +376,46 @@ def make_mafosun_checkpoint(cfg: Config, dtype: str = "bf16", seed: int = 1234, 
             for j in range(mo.experts):
                 sd[f"{p}.mlp.e{j}.gate"], sd[f"{p}.mlp.e{j}.up"], sd[f"{p}.mlp.e{j}.down"] = rn(mo.ff, H, s=4 * std), rn(mo.ff, H, s=4 * std), rn(H, mo.ff, s=4 * std)
     return sd
+
+
+def make_lilenex_checkpoint(cfg: Config, dtype: str = "bf16", seed: int = 1234, device="cpu", std: float = 0.05, router_std: float = 0.5) -> dict:
+    """Random weights of a Lilenex model under the names its checkpoints use: ``embed``, ``final.norm`` and per layer ``l<i>.{norm1, norm2}``,
+    ``l<i>.hc<q>.{in, out, mix}``, ``l<i>.mix.*`` and ``l<i>.mlp.*``."""
+    gen = torch.Generator(device=device)
+    gen.manual_seed(seed * 1000003 + 737371)
+    td, H = TORCH_DTYPES[dtype], cfg.hidden_size
+
+    def rn(*shape, s=std):
+        return (torch.randn(shape, generator=gen, device=device, dtype=torch.float32) * s).to(td)
+
+    def ru(*shape, lo=0.8, hi=1.2):
+        return (torch.rand(shape, generator=gen, device=device, dtype=torch.float32) * (hi - lo) + lo).to(td)
+
+    sd = {"embed": rn(cfg.vocab_size, H, s=1.0), "final.norm": ru(H)}
+    for i, sp in enumerate(cfg.layers):
+        p, n = cfg.layer_name(i), sp.streams
+        m, sq, mo = p + ".mix", sp.heads * sp.dim, sp.moe
+        sd[f"{m}.q"], sd[f"{m}.o"] = rn(sq, H, s=4 * std), rn(H, sp.inner, s=4 * std)
+        if sp.type == "sink_attention":
+            sd[f"{m}.q.norm"] = ru(sq, lo=0.5, hi=1.5)
+            if not sp.kv_back:
+                sd[f"{m}.k"], sd[f"{m}.v"] = rn(sp.n_kv * sp.dim, H, s=4 * std), rn(sp.n_kv * sp.vdim, H, s=4 * std)
+                sd[f"{m}.k.norm"] = ru(sp.n_kv * sp.dim, lo=0.5, hi=1.5)
+        else:
+            r = sp.decay_rank or 8
+            sd[f"{m}.k"], sd[f"{m}.v"], sd[f"{m}.g"] = rn(sq, H, s=4 * std), rn(sp.inner, H, s=4 * std), rn(sp.inner, H, s=4 * std)
+            sd[f"{m}.norm"], sd[f"{m}.a1"], sd[f"{m}.a2"], sd[f"{m}.a2.b"] = ru(sp.vdim), rn(r, H, s=4 * std), rn(sq, r, s=r ** -0.5), rn(sq, s=1.0)
+        if sp.dense_ff:
+            sd[f"{p}.mlp.up"], sd[f"{p}.mlp.down"] = rn(sp.dense_ff, H, s=4 * std), rn(H, sp.dense_ff, s=4 * std)
+        elif mo is not None:
+            sd[f"{p}.mlp.router"] = rn(mo.experts, H, s=router_std)
+            for j in range(mo.experts):
+                sd[f"{p}.mlp.e{j}.gate"], sd[f"{p}.mlp.e{j}.up"], sd[f"{p}.mlp.e{j}.down"] = rn(mo.ff, H, s=4 * std), rn(mo.ff, H, s=4 * std), rn(H, mo.ff, s=4 * std)
+            if mo.shared_ff:
+                for k, shape in (("gate", (mo.shared_ff, H)), ("up", (mo.shared_ff, H)), ("down", (H, mo.shared_ff))):
+                    sd[f"{p}.mlp.shared.{k}"] = rn(*shape, s=4 * std)
+        for q in (1, 2) if sp.dense_ff or mo is not None else (1,):
+            sd[f"{p}.norm{q}"] = ru(H)
+            sd[f"{p}.hc{q}.in"], sd[f"{p}.hc{q}.out"] = rn(n, s=0.5), ru(n, lo=0.5, hi=1.5)
+            sd[f"{p}.hc{q}.mix"] = (torch.eye(n, device=device) * 0.8 + torch.randn((n, n), generator=gen, device=device) * 0.2).to(td)
+    return sd

@@ -435,7 +435,7 @@ class _B200Session:
             raise ValueError(f"forward pass failed for layer {ops[0][0]} (block_idx={ops[0][2]}): activation dtype "
                              f"{x.dtype_name} != model dtype {be.dtype}")
         a = x.to_numpy_bits()
-        if a.ndim != 3 or a.shape[2] != ctx.config.hidden_size:
+        if a.ndim != 3 or a.shape[2] != ctx.config.stream_width:
             raise ValueError(f"forward pass failed for layer {ops[0][0]} (block_idx={ops[0][2]}): unexpected shape {x.shape}")
         a = np.ascontiguousarray(a)
         # consecutive ops that share index_pos go down in one call (they always do: text_model.rs:298-321)

@@ -84,6 +84,9 @@ typedef struct cake_b200_config {
   int layer_list;
   float logit_softcap;   /* logits <- cap * tanh(logits / cap) after the head (0 = none) */
   int scalar_final_norm; /* the final norm's gain is ONE number (ln_f points to a single element) instead of [hidden] */
+  int streams;           /* > 0: a token has that many residual streams (mixer-list blocks with spec.streams of the same number): x_dev / y_dev of
+                            cake_b200_forward_batch and the output of cake_b200_embed are (batch, seq, streams, hidden), all equal to the
+                            embedding at the start; the head reads their sum */
 } cake_b200_config;
 
 const char *cake_b200_last_error(void); /* thread-local; valid until the next call on this thread */
@@ -230,7 +233,14 @@ int cake_b200_block_load_spec(cake_b200_ctx *, int layer_idx, const cake_b200_la
  *                            uv; portions with key and value size 128 in 16-bit D expand k and v for the rows the step sees);
  *                            score = (q . k) * scale over the window (as above, keep_first included); head h's output is
  *                            multiplied by sigmoid(g h)_h (g [heads, hidden]; NULL = none); then o.
+ *   CAKE_B200_MIX_GATED_LINEAR  linear attention with a decay per key channel: q (times dim^-1/2), k [heads * dim, hidden], v [heads * vdim,
+ *                            hidden]; z = a2 (a1 h) + a2_b (a1 [decay_rank, hidden], a2 [heads * dim, decay_rank]), alpha =
+ *                            sigmoid(z)^(1 / decay_tau); S_t = diag(alpha_t) S_{t-1} + k_t v_t^T, o_t = S_t^T q_t; o of every head divided by
+ *                            its root mean square, times norm [vdim], times silu(g h), then o.  S lives in the cache in fp32.
  * Block structure switches (all 0 / NULL for the plain pre-norm block above):
+ *   streams      > 0: several residual streams X_s per token (cake_b200_config.streams).  A sublayer q (1 mixer, 2 feed-forward) reads
+ *                norm_q(sum_s in[s] X_s); with its output y, all streams at once: X_t <- sum_s mix[s, t] X_s + residual_mult out[t] y
+ *                (hc<q>_in, hc<q>_out [streams], hc<q>_mix [streams, streams])
  *   norm_kind    0: RMS norms; 1: the element-wise squashing norm tanh(alpha x) * w + b for norm1 / post1 / norm2 / post2, alpha =
  *                norm_alpha[0..3] in that order, offsets norm1_b / post1_b / norm2_b / post2_b ([hidden])
  *   side_dim     > 0: after the feed-forward the stream receives a per-layer token input: e = columns [side_col, side_col +
@@ -250,7 +260,9 @@ int cake_b200_block_load_spec(cake_b200_ctx *, int layer_idx, const cake_b200_la
  *                side mixer's spec / tensors use the mixer fields only.  Retention may be the main or the side mixer too
  *   dense_ff     > 0: a dense gated feed-forward of that width instead of the routed one (ff_gate, ff_up [dense_ff, hidden],
  *                ff_down [hidden, dense_ff]); dense_act 0 silu(g) u, 1 tanh-gelu(g) u, 2: g' = min(g, dense_limit), u' = clamp(u,
- *                -dense_limit, dense_limit), g' sigmoid(1.702 g') (u' + 1), 3: max(g, 0) u */
+ *                -dense_limit, dense_limit), g' sigmoid(1.702 g') (u' + 1), 3: max(g, 0) u.  ff_gate NULL: ff_down act(ff_up h) without a
+ *                gate, act 0 silu, 1 tanh-gelu, 3 relu
+ *   A shared expert without s_sg is added as it is. */
 #define CAKE_B200_MIX_LATENT 1
 #define CAKE_B200_MIX_RETENTION 2
 #define CAKE_B200_MIX_STATE_SPACE 3
@@ -259,6 +271,7 @@ int cake_b200_block_load_spec(cake_b200_ctx *, int layer_idx, const cake_b200_la
 #define CAKE_B200_MIX_MATRIX_MEMORY 6
 #define CAKE_B200_MIX_SINK_ATTENTION 7
 #define CAKE_B200_MIX_LATENT_WINDOW 8
+#define CAKE_B200_MIX_GATED_LINEAR 9
 typedef struct cake_b200_rotary_spec {
   int dims;            /* 0 = no rotation */
   double base;
@@ -281,6 +294,8 @@ typedef struct cake_b200_moe_spec {
   int groups, groups_keep; /* groups > 1: the experts form that many equal groups of neighbours; only experts of the groups_keep groups with
                               the largest best score may be chosen */
   int plain_weights;       /* 1: the weights are the chosen experts' scores (times scale), not renormalised */
+  int sigmoid_scores;      /* 1: scores are sigmoid(logit) instead of a softmax over all experts */
+  int weigh_input;         /* 1: a chosen expert reads weight * h and its output is added as it is (no identity experts) */
 } cake_b200_moe_spec;
 typedef struct cake_b200_mixer_spec {
   int kind;
@@ -311,9 +326,16 @@ typedef struct cake_b200_mixer_spec {
   int chunk;              /* > 0: row i sees the keys of its own chunk of that many positions, counted from position 0 */
   float softcap;          /* > 0: score <- softcap * tanh(score / softcap) */
   int sink_zero;          /* 1: the denominator holds one more term exp(0) without a value */
-  int qk_norm;            /* 1: RMS norm of every q and k head with the gains q_norm / k_norm [dim], in front of the rotation */
+  int qk_norm;            /* 1: RMS norm of every q and k head with the gains q_norm / k_norm [dim], in front of the rotation; 2: one RMS norm over
+                             the whole q (k) projection with gains [heads * dim] ([kv_heads * dim]) */
   int v_unit;             /* 1: every value head is divided by its root mean square before it is cached */
   float branch_scale;     /* with a side mixer and without branch norms: y = branch_scale * main + side->branch_scale * side */
+  int kv_back;            /* sink attention: > 0: no keys and values of its own; reads those cached under block_idx - kv_back (same kv_heads,
+                             dim and vdim), which has run the step's positions before this block does */
+  int decay_rank;         /* gated linear */
+  float decay_tau;
+  int streams;            /* block structure: residual streams (0 = one stream, plain sums) */
+  float residual_mult;
 } cake_b200_mixer_spec;
 typedef struct cake_b200_mixer_tensors {
   const void *norm1, *norm2;                 /* [hidden]; norm2 NULL without a feed-forward */
@@ -334,7 +356,10 @@ typedef struct cake_b200_mixer_tensors {
   const void *dq, *dq_norm, *uq;             /* windowed latent attention: [q_rank, hidden], [q_rank], [heads * dim, q_rank] */
   const void *norm1_b, *post1_b, *norm2_b, *post2_b;  /* norm_kind 1: [hidden] each */
   const void *side_gate, *side_proj, *side_norm;      /* side_dim > 0: [side_dim, hidden], [hidden, side_dim], [hidden] */
-  const void *q_norm, *k_norm;               /* qk_norm: [dim] each */
+  const void *q_norm, *k_norm;               /* qk_norm 1: [dim] each; 2: [heads * dim], [kv_heads * dim] (k_norm NULL with kv_back) */
+  const void *a1, *a2, *a2_b;                /* gated linear: [decay_rank, hidden], [heads * dim, decay_rank], [heads * dim] */
+  const void *hc1_in, *hc1_out, *hc1_mix;    /* streams > 0: [streams], [streams], [streams (from), streams (to)] */
+  const void *hc2_in, *hc2_out, *hc2_mix;
 } cake_b200_mixer_tensors;
 int cake_b200_block_load_mixer(cake_b200_ctx *, int layer_idx, const cake_b200_mixer_spec *, const cake_b200_mixer_tensors *,
                                cake_b200_block **out);

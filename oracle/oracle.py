@@ -21,7 +21,7 @@ _SO = os.path.join(_HERE, "_build", "libcake_oracle.so")
 
 # ora_config mirrors the Llama-family prefix of cake_b200_config; the layer-list fields behind it have their own oracle
 # (oracle/nigenex_plain.py)
-_ORA_FIELDS = [f for f in CConfig._fields_ if f[0] not in ("layer_list", "logit_softcap", "scalar_final_norm")]
+_ORA_FIELDS = [f for f in CConfig._fields_ if f[0] not in ("layer_list", "logit_softcap", "scalar_final_norm", "streams")]
 
 
 class OraConfig(ctypes.Structure):

@@ -22,6 +22,7 @@ pub struct cake_b200_config {
     pub pre_reshape_qk_norm: c_int, // config.rs:116 (OLMo2)
     // layer-list models (per-layer geometry, fp32 residual stream): not a reference architecture, zero for cake's own models
     pub layer_list: c_int, pub logit_softcap: f32, pub scalar_final_norm: c_int,
+    pub streams: c_int,
 }
 
 /// `cake_b200_layer_spec` / `cake_b200_layer_tensors` (include/cake_b200.h): one layer of a layer-list model.
@@ -163,6 +164,8 @@ pub struct cake_b200_moe_spec {
     pub groups: c_int,
     pub groups_keep: c_int,
     pub plain_weights: c_int,
+    pub sigmoid_scores: c_int,
+    pub weigh_input: c_int,
 }
 #[repr(C)]
 pub struct cake_b200_mixer_spec {
@@ -208,6 +211,12 @@ pub struct cake_b200_mixer_spec {
     pub qk_norm: c_int,
     pub v_unit: c_int,
     pub branch_scale: f32,
+    // shared keys and values, gated linear attention, residual streams
+    pub kv_back: c_int,
+    pub decay_rank: c_int,
+    pub decay_tau: f32,
+    pub streams: c_int,
+    pub residual_mult: f32,
 }
 #[repr(C)]
 pub struct cake_b200_mixer_tensors {
@@ -274,6 +283,15 @@ pub struct cake_b200_mixer_tensors {
     pub side_norm: *const c_void,
     pub q_norm: *const c_void,
     pub k_norm: *const c_void,
+    pub a1: *const c_void,
+    pub a2: *const c_void,
+    pub a2_b: *const c_void,
+    pub hc1_in: *const c_void,
+    pub hc1_out: *const c_void,
+    pub hc1_mix: *const c_void,
+    pub hc2_in: *const c_void,
+    pub hc2_out: *const c_void,
+    pub hc2_mix: *const c_void,
 }
 
 /// `cake_b200_block_variant` (include/cake_b200.h): norm placement and per-layer attention mode of the OLMo2 / Gemma3 /
