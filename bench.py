@@ -12,6 +12,7 @@ Llama-3-8B bf16, bs=1, 2k context, layers sharded over N GPUs of one box (N=1 ->
     python bench.py --workload nuvarax [--sizes 1k,2k]            # the Nuvarax design beside the closest existing model
     python bench.py --workload netolorn [--sizes 1k,2k]           # the Netolorn design beside the closest existing models
     python bench.py --workload mafosun [--sizes 1k,2k]            # the Mafosun design beside the closest existing models
+    python bench.py --workload lilenex [--sizes 1k,2k]            # the Lilenex design beside the closest existing models
 
 A "step" is one decoded token: one pass of the hot path (embed -> blocks -> ln_f/lm_head/argmax) at batch 1.
 tok/s follows the reference's definition (master.rs:131-166): prefill excluded.  Prints ONE JSON line (rank 0).
@@ -1492,6 +1493,104 @@ def mafosun_leg(env: Env, sizes=("1k", "2k"), batch: int = 4, seq: int = 4096, c
             "peaks": {"tensor_tflops": pk["tc"], "hbm_gbs": pk["hbm"], "source": pk["src"]}, "sizes": out}
 
 
+LILENEX_SIZES = {
+    "1k": dict(width=1024, streams=4, ff=4096, window=1024, keep_first=4, att=dict(heads=8, kv_heads=2, dim=128, vdim=128, rot_dims=64),
+               gla=dict(heads=4, dim=128, vdim=128), rank=16, moe=dict(experts=32, top=4, ff=704, shared_ff=704)),
+    "2k": dict(width=2048, streams=4, ff=8192, window=1024, keep_first=4, att=dict(heads=16, kv_heads=4, dim=128, vdim=128, rot_dims=64),
+               gla=dict(heads=8, dim=128, vdim=128), rank=16, moe=dict(experts=64, top=6, ff=1408, shared_ff=1408)),
+}
+
+
+def lilenex_leg(env: Env, sizes=("1k", "2k"), batch: int = 4, seq: int = 4096, ctx_len: int = 2048, steps: int = 32, reps: int = 3) -> dict:
+    """`--workload lilenex`: the Lilenex design (mixer-list blocks with several residual streams) in three 4-layer models per size, two of
+    them beside the framework's closest existing model at equal width:
+      attention   4 x (grouped-query attention with a window that keeps the first tokens, norms over the whole q / k projections, a partial
+                  rotation + dense feed-forward without a gate)  beside the Netolorn attention layer (window, kept tokens, sink, gate; gated dense)
+      linear      4 x (gated linear attention with a decay per key channel + routed feed-forward with a shared expert)  beside four Setodra
+                  retention layers with a routed feed-forward of the same sizes
+      mixed       linear + dense, attention + routed, attention that shares its keys + routed, linear + routed (the headline; no counterpart)
+    all through TextModelBase / forward_batch.  Workload and timing as in the Setodra leg."""
+    import torch
+    from cake_b200.config import Config, MixerSpec, MoeSpec, RotarySpec
+    from cake_b200.synth import make_lilenex_checkpoint, make_mixer_checkpoint, make_netolorn_checkpoint
+    pk = peaks()
+    out, launches, vocab = {}, 0, 32768
+    mseq = max(seq, ctx_len + steps + 8)
+    for name in sizes:
+        z = LILENEX_SIZES[name]
+        W, ff, win, keep, a, g, mo, ns, rank = z["width"], z["ff"], z["window"], z["keep_first"], z["att"], z["gla"], z["moe"], z["streams"], z["rank"]
+        H, G, D, V = a["heads"], a["kv_heads"], a["dim"], a["vdim"]
+        dense_ff = {"kind": "dense", "ff": ff}
+        routed = {"kind": "moe", "router": {"experts": mo["experts"], "top": mo["top"]}, "expert": {"ff": mo["ff"]}, "shared": {"ff": mo["shared_ff"]}}
+        rot = {"dims": a["rot_dims"], "base": 10000.0, "scaling": {"factor": 8.0, "original": 2048, "fast": 32.0, "slow": 1.0}}
+        att = {"heads": H, "kv_heads": G, "dim": D, "vdim": V, "scale": D ** -0.5, "mask": {"size": win, "keep_first": keep}, "rot": rot}
+        lin = dict(g, tau=16.0)
+        orders = {"attention": [("attention", att, dense_ff)] * 4, "linear": [("gla", lin, routed)] * 4,
+                  "mixed": [("gla", lin, dense_ff), ("attention", att, routed), ("attention", dict(att, kv_from=1), routed), ("gla", lin, routed)]}
+        # algorithmic work per token: products [flops = bytes of weights read by one decoded token], attended keys, state updates, cache rows
+        keys = lambda S: sum(min(i + 1, win + keep) for i in range(S))
+        hd, hv = g["heads"] * g["dim"], g["heads"] * g["vdim"]
+        lin_q, lin_kv, lin_gla = 2.0 * W * (H * D + H * V), 2.0 * W * G * (D + V), 2.0 * W * (2 * hd + 3 * hv + rank) + 2.0 * rank * hd
+        lin_ff = {"dense": 2.0 * W * 2 * ff, "moe": 2.0 * W * 3 * (mo["top"] * mo["ff"] + mo["shared_ff"]) + 2.0 * W * mo["experts"]}
+        state = 4.0 * g["heads"] * g["dim"] * g["vdim"]
+        row = {"size": z}
+        for arch in ("attention", "attention_closest", "linear", "linear_closest", "mixed"):
+            if arch in orders:
+                order = [{"type": t, "mixer": m, "mlp": f} for t, m, f in orders[arch]]
+                cfg = Config.from_hf({"architecture": "Lilenex", "width": W, "vocab": vocab, "norm": {"eps": 1e-6}, "streams": ns, "residual_mult": 0.7, "layers": order})
+                for sp in cfg.layers:
+                    sp.decay_rank = rank if sp.type == "gated_linear" else 0
+                sd = make_lilenex_checkpoint(cfg, "bf16", seed=5, device=env.dev, std=0.01)
+                n_att = sum(1 for L in order if L["type"] == "attention")
+                n_kv = sum(1 for L in order if L["type"] == "attention" and "kv_from" not in L["mixer"])
+                flop_tok = n_att * lin_q + n_kv * lin_kv + (4 - n_att) * lin_gla + sum(lin_ff[L["mlp"]["kind"]] for L in order)
+                att_flops = n_att * 2.0 * H * (D + V) * keys(seq) + (4 - n_att) * state * seq
+                dbytes = flop_tok + n_att * 2.0 * G * (D + V) * (min(win, ctx_len) + keep) + (4 - n_att) * 2.0 * state
+            elif arch == "attention_closest":
+                L = {"type": "attention", "mlp": dense_ff, "mixer": att}
+                cfg = Config.from_hf({"architecture": "Netolorn", "width": W, "vocab": vocab, "norm": {"eps": 1e-6}, "layers": [L] * 4})
+                sd = make_netolorn_checkpoint(cfg, "bf16", seed=5, device=env.dev, std=0.02)
+                flop_tok = 4 * (lin_q + lin_kv + 2.0 * W * H * V + 2.0 * W * 3 * ff)
+                att_flops = 4 * 2.0 * H * (D + V) * keys(seq)
+                dbytes = flop_tok + 4 * 2.0 * G * (D + V) * (min(win, ctx_len) + keep)
+            else:
+                m = MoeSpec(scale=2.5, experts=mo["experts"], identity=0, top=mo["top"], ff=mo["ff"], shared_ff=mo["shared_ff"])
+                decay = [1.0 - 2.0 ** -(5 + i * 5.0 / g["heads"]) for i in range(g["heads"])]
+                spec = MixerSpec(type="retention", heads=g["heads"], dim=g["dim"], vdim=g["vdim"], decay=decay, rot=RotarySpec(dims=g["dim"], base=10000.0), moe=m)
+                cfg = Config(hidden_size=W, intermediate_size=0, vocab_size=vocab, num_hidden_layers=4, num_attention_heads=g["heads"],
+                             num_key_value_heads=g["heads"], rms_norm_eps=1e-6, head_dim=g["vdim"], max_seq_len=mseq, block_kind="setodra", layers=[spec] * 4,
+                             model_prefix="", embed_scale=1.0)
+                sd = make_mixer_checkpoint(cfg, "bf16", seed=5, device=env.dev, std=0.02)
+                flop_tok = 4 * (2.0 * W * (2 * hd + 3 * hv) + lin_ff["moe"])
+                att_flops = 4 * state * seq
+                dbytes = flop_tok + 4 * 2.0 * state
+            cfg.max_seq_len = mseq
+            t = _time_listed_model(env, cfg, sd, batch, seq, ctx_len, steps, reps, mseq)
+            del sd
+            torch.cuda.empty_cache()
+            launches += t["launches"]
+            M, ms, dms = batch * seq, t["prefill"]["ms"], t["decode"]["ms_per_token"]
+            flops = flop_tok * M + batch * att_flops + 2.0 * batch * vocab * W
+            dbytes += 2.0 * vocab * W
+            row[arch] = {"prefill": {"tok_s": M / (ms / 1e3), "ms": ms, "tflops": flops / (ms * 1e-3) / 1e12,
+                                     "frac_of_tensor_peak": flops / (ms * 1e-3) / 1e12 / pk["tc"], "finite": t["prefill"]["finite"],
+                                     "launches": t["prefill"]["launches"]},
+                         "decode": {"tok_s": 1e3 / dms, "ms_per_token": dms, "gb_s": dbytes / (dms * 1e-3) / 1e9,
+                                    "frac_of_hbm_peak": dbytes / (dms * 1e-3) / 1e9 / pk["hbm"], "launches_per_token": t["decode"]["launches_per_token"],
+                                    "finite": t["decode"]["finite"]}}
+        for kind in ("attention", "linear"):   # how far from the roofline each is, the new design over the closest model (1 = equally far)
+            row[kind + "_prefill_distance"] = row[kind + "_closest"]["prefill"]["frac_of_tensor_peak"] / row[kind]["prefill"]["frac_of_tensor_peak"]
+            row[kind + "_decode_distance"] = row[kind + "_closest"]["decode"]["frac_of_hbm_peak"] / row[kind]["decode"]["frac_of_hbm_peak"]
+        out[name] = row
+    head = out[sizes[-1]]
+    return {"metric": f"lilenex prefill tok/s (4 layers, width {head['size']['width']}, bf16, bs={batch} x {seq})", "value": head["mixed"]["prefill"]["tok_s"],
+            "unit": "tok/s", "ms_per_step": head["mixed"]["prefill"]["ms"], "steps": reps, "warmup": 1, "gpu_launches": int(launches),
+            "config": {"workload": f"Lilenex (attention / linear / mixed layer orders) vs the Netolorn attention layer and the Setodra retention layer at equal width, "
+                                   f"4 layers, bf16, prefill bs={batch} x {seq}, decode bs=1 at {ctx_len} context x {steps} steps",
+                       "l2": "prefill activations / decode weights exceed L2"},
+            "peaks": {"tensor_tflops": pk["tc"], "hbm_gbs": pk["hbm"], "source": pk["src"]}, "sizes": out}
+
+
 # ------------------------------------------------------------------------------------------------
 def run_cuda(args):
     env = Env(args)
@@ -1527,12 +1626,12 @@ def run_cuda(args):
             line.update({"n_gpus": 1, "higher_is_better": True, "scaling": "strong", "vs_baseline": None, "dtype": "bf16", "data": "synthetic"})
             emit(line)
         return
-    if args.workload in ("netolorn", "mafosun"):
+    if args.workload in ("netolorn", "mafosun", "lilenex"):
         if rank == 0:
             if env.sampler:
                 env.sampler.start()
             sizes = tuple((args.sizes if args.sizes != "2k,4k,4k-hd64" else "1k,2k").split(","))
-            leg = netolorn_leg if args.workload == "netolorn" else mafosun_leg
+            leg = {"netolorn": netolorn_leg, "mafosun": mafosun_leg, "lilenex": lilenex_leg}[args.workload]
             line = leg(env, sizes=sizes, batch=args.pf_batch, seq=args.pf_seq, steps=max(4, min(args.steps, 64)))
             line["clocks"] = env.sampler.stop() if env.sampler else None
             line.update({"n_gpus": 1, "higher_is_better": True, "scaling": "strong", "vs_baseline": None, "dtype": "bf16", "data": "synthetic"})
@@ -1611,9 +1710,9 @@ def main():
     ap.add_argument("--warmup", type=int, default=8)
     ap.add_argument("--impl", default="cuda", choices=["cuda", "reference"])
     ap.add_argument("--model", default="8b", choices=["8b", "70b"])
-    ap.add_argument("--workload", default="decode", choices=["decode", "prefill", "nigenex", "setodra", "nuvarax", "netolorn", "mafosun"])
-    ap.add_argument("--pf-batch", type=int, default=4, help="--workload setodra / nuvarax / netolorn / mafosun: batch rows of the prefill step")
-    ap.add_argument("--pf-seq", type=int, default=4096, help="--workload setodra / nuvarax / netolorn / mafosun: tokens per row of the prefill step")
+    ap.add_argument("--workload", default="decode", choices=["decode", "prefill", "nigenex", "setodra", "nuvarax", "netolorn", "mafosun", "lilenex"])
+    ap.add_argument("--pf-batch", type=int, default=4, help="--workload setodra / nuvarax / netolorn / mafosun / lilenex: batch rows of the prefill step")
+    ap.add_argument("--pf-seq", type=int, default=4096, help="--workload setodra / nuvarax / netolorn / mafosun / lilenex: tokens per row of the prefill step")
     ap.add_argument("--sizes", default="2k,4k,4k-hd64", help="--workload nigenex: which of NIGENEX_SIZES to run")
     ap.add_argument("--extras", default="auto", choices=["auto", "none", "all"],
                     help="auto: config0 + config4 at N=1, config3 (70B) at N=8; none: the headline only")

@@ -1118,6 +1118,16 @@ __global__ void __launch_bounds__(128) moe_gather_kernel(const T *__restrict__ h
   constexpr int VE = 16 / (int)sizeof(T);
   if (wts && src) {
     const float w = wts[e];
+    if (sizeof(T) == 2 && W % 8 == 0) {
+      typedef typename Bits16<T>::type B;
+      for (int i = threadIdx.x; i < W / 8; i += blockDim.x) {
+        float v[8];
+        unpack8<B>(reinterpret_cast<const uint4 *>(src)[i], v);
+        reinterpret_cast<uint4 *>(dst)[i] = make_uint4(pack2x<B>(w * v[0], w * v[1]), pack2x<B>(w * v[2], w * v[3]), pack2x<B>(w * v[4], w * v[5]),
+                                                       pack2x<B>(w * v[6], w * v[7]));
+      }
+      return;
+    }
     if (W % 4 == 0) {
       for (int i = threadIdx.x; i < W / 4; i += blockDim.x) {
         float v[4];

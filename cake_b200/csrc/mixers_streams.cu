@@ -24,8 +24,6 @@ namespace mx {
     return (int)cudaGetLastError();    \
   } while (0)
 
-__device__ __forceinline__ float softplus_f(float z) { return fmaxf(z, 0.f) + log1pf(expf(-fabsf(z))); }
-
 template <typename T> __device__ __forceinline__ void load4(const T *s, float (&v)[4]) {
   const uint2 u = *reinterpret_cast<const uint2 *>(s);
   const float2 a = DT<T>::unpack2(u.x), b = DT<T>::unpack2(u.y);
@@ -244,10 +242,11 @@ __global__ void __launch_bounds__(128) channel_decay_kernel(const ChannelDecay p
       z[t] = fmaf(wj, u.x, z[t]); z[t + 1] = fmaf(wj, u.y, z[t + 1]); z[t + 2] = fmaf(wj, u.z, z[t + 2]); z[t + 3] = fmaf(wj, u.w, z[t + 3]);
     }
   }
-  // sigmoid(z)^(1 / tau) = exp(-softplus(-z) / tau)
+  // sigmoid(z)^(1 / tau) = exp(-softplus(-z) / tau); the rounding of 1 + exp(-|z|) moves the result by less than its last place / tau
+  const float itau = 1.0f / p.tau;
 #pragma unroll
   for (int t = 0; t < CD_TT; t++)
-    if (t < nt) p.a[(size_t)(m0 + t) * p.channels + ch] = expf(-softplus_f(-z[t]) / p.tau);
+    if (t < nt) p.a[(size_t)(m0 + t) * p.channels + ch] = expf(-(fmaxf(-z[t], 0.f) + logf(1.0f + expf(-fabsf(z[t])))) * itau);
 }
 int channel_decay(cudaStream_t st, int dtype, const ChannelDecay &p, uint64_t *launches) {
   if (p.M < 1 || p.channels < 1 || p.rank < 1 || !(p.tau > 0.f)) return (int)cudaErrorInvalidValue;
@@ -266,25 +265,28 @@ int channel_decay(cudaStream_t st, int dtype, const ChannelDecay &p, uint64_t *l
 // ---------------------------------------------------------------------------------------------- recurrence with channel decays
 // A CTA walks the step's tokens for CW * 16 columns of one (head, batch row)'s state.  Its eight warps are RW row groups of 32 key
 // channels by CW column groups of 16; a lane keeps a 4 x 4 tile of the state in registers (lane & 7: which four rows, lane >> 3: which
-// four columns), so that a token costs it four 16-byte shared-memory loads (q, k, a of its rows, v of its columns) for 48 multiply-adds.
-// Tokens come in chunks of 16: the raw values of the next chunk wait in registers while the current one is computed; the partial
-// outputs of a warp's rows are summed over its lanes by a transposing exchange, those of the row groups once per chunk.  Rows
-// beyond dk and columns beyond dv hold zeros.
-constexpr int CR_TT = 16;
-template <typename T> struct Raw4 { typedef uint2 type; };
-template <> struct Raw4<float> { typedef float4 type; };
-template <typename T> __device__ __forceinline__ float4 raw_to_f4(const typename Raw4<T>::type &r) {
-  const float2 a = DT<T>::unpack2(r.x), b = DT<T>::unpack2(r.y);
-  return make_float4(a.x, a.y, b.x, b.y);
+// four columns), so that a token costs it four shared-memory loads (q, k, a of its rows, v of its columns) for 48 multiply-adds.
+// Tokens come in chunks of CR_TT, copied asynchronously as they are (q, k, v in D, a in fp32) into one of two buffers while the other is
+// computed on; the partial outputs of a warp's rows are summed over its lanes by a transposing exchange, those of the row groups
+// once per chunk.  Rows beyond dk and columns beyond dv hold zeros; places behind the step's last token leave the state as it is.
+constexpr int CR_TT = 32;
+template <typename T, int RW> struct ChannelTile {
+  static constexpr int CW = 8 / RW, DK = RW * 32, CB = CW * 16;
+  static constexpr int STAGE = CR_TT * (DK * (2 * (int)sizeof(T) + 4) + CB * (int)sizeof(T));  // a, q, k, v of a chunk in bytes
+  static constexpr int SMEM = 2 * STAGE + RW * CR_TT * CB * 4;
+};
+// four entries global -> shared (8 bytes in 16-bit D, 16 in fp32); nothing is read and zeros arrive when !in
+template <int BYTES> __device__ __forceinline__ void copy_async(void *dst, const void *src, bool in) {
+  const int n = in ? BYTES : 0;
+  asm volatile("cp.async.ca.shared.global [%0], [%1], %2, %3;" ::"r"(smem_u32(dst)), "l"(src), "n"(BYTES), "r"(n) : "memory");
 }
-template <> __device__ __forceinline__ float4 raw_to_f4<float>(const float4 &r) { return r; }
 
 template <typename T, int RW>
-__global__ void __launch_bounds__(256) recurrence_channels_kernel(const Recurrence p) {
-  constexpr int CW = 8 / RW, DK = RW * 32, CB = CW * 16, NQ = (CR_TT * DK / 4 + 255) / 256;  // NQ: 4-entry pieces of q (k, a) per thread and chunk
-  constexpr int NVP = (CR_TT * CB / 4 + 255) / 256;
-  extern __shared__ __align__(16) float sm[];
-  float *qs = sm, *ks = qs + CR_TT * DK, *as = ks + CR_TT * DK, *vs = as + CR_TT * DK, *part = vs + CR_TT * CB;  // part [RW][CR_TT][CB]
+__global__ void __launch_bounds__(256, 1) recurrence_channels_kernel(const Recurrence p) {
+  typedef ChannelTile<T, RW> C;
+  constexpr int DK = C::DK, CB = C::CB, PB = 4 * (int)sizeof(T);
+  extern __shared__ __align__(16) unsigned char raw[];
+  float *part = reinterpret_cast<float *>(raw + 2 * C::STAGE);  // [RW][CR_TT][CB]
   const int ncb = (p.dv + CB - 1) / CB, h = blockIdx.x / ncb, c0 = (blockIdx.x % ncb) * CB, b = blockIdx.y;
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, rw = warp % RW, cw = warp / RW;
   const int rl = lane & 7, cl = lane >> 3, row0 = rw * 32 + rl * 4, colb = cw * 16 + cl * 4, col0 = c0 + colb;
@@ -297,88 +299,79 @@ __global__ void __launch_bounds__(256) recurrence_channels_kernel(const Recurren
     if (live && p.pos0 > 0) s = *reinterpret_cast<const float4 *>(gs + (size_t)r * p.dv);
     St[r][0] = s.x; St[r][1] = s.y; St[r][2] = s.z; St[r][3] = s.w;
   }
-  typedef typename Raw4<T>::type R4;
-  R4 rq[NQ], rk[NQ], rv[NVP];
-  float4 ra[NQ];
-  const int dk4 = p.dk / 4, dv4 = p.dv / 4;
-  auto fetch = [&](int t0) {  // indices are clamped: what lies beyond the chunk or the head is replaced when the chunk is staged
+  auto fetch = [&](int t0, int stage) {
     const int nt = min(CR_TT, p.S - t0);
     const size_t m0 = (size_t)b * p.S + t0;
+    float *as = reinterpret_cast<float *>(raw + stage * C::STAGE);
+    T *qs = reinterpret_cast<T *>(as + CR_TT * DK), *ks = qs + CR_TT * DK, *vs = ks + CR_TT * DK;
+    for (int idx = threadIdx.x; idx < CR_TT * DK / 4; idx += 256) {
+      const int tt = idx / (DK / 4), i = 4 * (idx % (DK / 4));
+      const bool in = tt < nt && i < p.dk;
+      const size_t m = in ? m0 + tt : m0;
+      const int e = h * p.dk + (in ? i : 0);
+      copy_async<PB>(qs + 4 * idx, reinterpret_cast<const T *>(p.q) + m * p.ldq + e, in);
+      copy_async<PB>(ks + 4 * idx, reinterpret_cast<const T *>(p.k) + m * p.ldk + e, in);
+      if (tt < nt) copy_async<16>(as + 4 * idx, p.a_chan + m * p.heads * p.dk + e, in);
+      else *reinterpret_cast<float4 *>(as + 4 * idx) = make_float4(1.f, 1.f, 1.f, 1.f);
+    }
+    for (int idx = threadIdx.x; idx < CR_TT * CB / 4; idx += 256) {
+      const int tt = idx / (CB / 4), i = c0 + 4 * (idx % (CB / 4));
+      const bool in = tt < nt && i < p.dv;
+      copy_async<PB>(vs + 4 * idx, reinterpret_cast<const T *>(p.v) + (in ? m0 + tt : m0) * p.ldv + (size_t)h * p.dv + (in ? i : 0), in);
+    }
+    asm volatile("cp.async.commit_group;" ::: "memory");
+  };
+  const bool b0 = rl & 1, b1 = rl & 2, b2 = rl & 4;
+  // Four tokens at a time: their operands are loaded ahead of the updates, their 16 partial outputs (token j, column c at 4 j + c) are
+  // summed over the eight lanes that share the columns by exchanges that halve what a lane holds: 8 + 4 + 2 shuffles leave it the
+  // two sums of token 2 b0 + b1, columns 2 b2 and 2 b2 + 1 (b0, b1, b2: the bits of rl).
+  auto four = [&](const float *as, const T *qs, const T *ks, const T *vs, int t4) {
+    float q[4][4], k[4][4], a[4][4], v[4][4], x[16];
 #pragma unroll
-    for (int e = 0; e < NQ; e++) {
-      const int idx = threadIdx.x + 256 * e, tt = min(idx / (DK / 4), nt - 1), i = min(idx % (DK / 4), dk4 - 1);
-      rq[e] = *reinterpret_cast<const R4 *>(reinterpret_cast<const T *>(p.q) + (m0 + tt) * p.ldq + (size_t)h * p.dk + 4 * i);
-      rk[e] = *reinterpret_cast<const R4 *>(reinterpret_cast<const T *>(p.k) + (m0 + tt) * p.ldk + (size_t)h * p.dk + 4 * i);
-      ra[e] = *reinterpret_cast<const float4 *>(p.a_chan + ((m0 + tt) * p.heads + h) * p.dk + 4 * i);
+    for (int j = 0; j < 4; j++) {
+      load4<T>(qs + (t4 + j) * DK + row0, q[j]);
+      load4<T>(ks + (t4 + j) * DK + row0, k[j]);
+      load4<float>(as + (t4 + j) * DK + row0, a[j]);
+      load4<T>(vs + (t4 + j) * CB + colb, v[j]);
     }
 #pragma unroll
-    for (int e = 0; e < NVP; e++) {
-      const int idx = threadIdx.x + 256 * e, tt = min(idx / (CB / 4), nt - 1), i = min(c0 / 4 + idx % (CB / 4), dv4 - 1);
-      rv[e] = *reinterpret_cast<const R4 *>(reinterpret_cast<const T *>(p.v) + (m0 + tt) * p.ldv + (size_t)h * p.dv + 4 * i);
+    for (int j = 0; j < 4; j++) {
+#pragma unroll
+      for (int c = 0; c < 4; c++) x[4 * j + c] = 0.f;
+#pragma unroll
+      for (int r = 0; r < 4; r++)
+#pragma unroll
+        for (int c = 0; c < 4; c++) {
+          St[r][c] = fmaf(a[j][r], St[r][c], k[j][r] * v[j][c]);
+          x[4 * j + c] = fmaf(St[r][c], q[j][r], x[4 * j + c]);
+        }
     }
-  };
-  const bool hi1 = rl & 1, hi2 = rl & 2;
-  const int pcol = colb + (rl & 1) * 2 + ((rl >> 1) & 1);  // the column whose sum this lane ends up with
-  auto token = [&](int tt) {
-    const float4 q = *reinterpret_cast<const float4 *>(qs + tt * DK + row0), k = *reinterpret_cast<const float4 *>(ks + tt * DK + row0);
-    const float4 a = *reinterpret_cast<const float4 *>(as + tt * DK + row0), v = *reinterpret_cast<const float4 *>(vs + tt * CB + colb);
-    const float qr[4] = {q.x, q.y, q.z, q.w}, kr[4] = {k.x, k.y, k.z, k.w}, ar[4] = {a.x, a.y, a.z, a.w}, vc[4] = {v.x, v.y, v.z, v.w};
-    float acc[4] = {0.f, 0.f, 0.f, 0.f};
+    float y[8], z[4], o[2];
 #pragma unroll
-    for (int r = 0; r < 4; r++)
+    for (int i = 0; i < 8; i++) y[i] = (b0 ? x[8 + i] : x[i]) + __shfl_xor_sync(0xffffffffu, b0 ? x[i] : x[8 + i], 1);
 #pragma unroll
-      for (int c = 0; c < 4; c++) {
-        St[r][c] = fmaf(ar[r], St[r][c], kr[r] * vc[c]);
-        acc[c] = fmaf(St[r][c], qr[r], acc[c]);
-      }
-    // lanes that differ in rl share columns: two exchanges halve the columns a lane holds, the third adds the rest
-    float k0 = hi1 ? acc[2] : acc[0], k1 = hi1 ? acc[3] : acc[1];
-    k0 += __shfl_xor_sync(0xffffffffu, hi1 ? acc[0] : acc[2], 1);
-    k1 += __shfl_xor_sync(0xffffffffu, hi1 ? acc[1] : acc[3], 1);
-    float s = hi2 ? k1 : k0;
-    s += __shfl_xor_sync(0xffffffffu, hi2 ? k0 : k1, 2);
-    s += __shfl_xor_sync(0xffffffffu, s, 4);
-    if (rl < 4) part[(rw * CR_TT + tt) * CB + pcol] = s;
+    for (int i = 0; i < 4; i++) z[i] = (b1 ? y[4 + i] : y[i]) + __shfl_xor_sync(0xffffffffu, b1 ? y[i] : y[4 + i], 2);
+#pragma unroll
+    for (int i = 0; i < 2; i++) o[i] = (b2 ? z[2 + i] : z[i]) + __shfl_xor_sync(0xffffffffu, b2 ? z[i] : z[2 + i], 4);
+    *reinterpret_cast<float2 *>(part + (rw * CR_TT + t4 + 2 * b0 + b1) * CB + colb + 2 * b2) = make_float2(o[0], o[1]);
   };
-  fetch(0);
-  for (int t0 = 0; t0 < p.S; t0 += CR_TT) {
+  fetch(0, 0);
+  for (int t0 = 0, stage = 0; t0 < p.S; t0 += CR_TT, stage ^= 1) {
     const int nt = min(CR_TT, p.S - t0);
     const size_t m0 = (size_t)b * p.S + t0;
-    __syncthreads();  // the previous chunk's outputs have been added up
-#pragma unroll
-    for (int e = 0; e < NQ; e++) {
-      const int idx = threadIdx.x + 256 * e;
-      const bool in = idx % (DK / 4) < dk4;
-      float4 q = raw_to_f4<T>(rq[e]), k = raw_to_f4<T>(rk[e]), a = ra[e];
-      q.x *= p.qscale; q.y *= p.qscale; q.z *= p.qscale; q.w *= p.qscale;
-      k.x *= p.kscale; k.y *= p.kscale; k.z *= p.kscale; k.w *= p.kscale;
-      if (!in) q = k = a = make_float4(0.f, 0.f, 0.f, 0.f);
-      if (idx >= CR_TT * DK / 4) continue;
-      reinterpret_cast<float4 *>(qs)[idx] = q;
-      reinterpret_cast<float4 *>(ks)[idx] = k;
-      reinterpret_cast<float4 *>(as)[idx] = a;
-    }
-#pragma unroll
-    for (int e = 0; e < NVP; e++) {
-      const int idx = threadIdx.x + 256 * e;
-      if (idx < CR_TT * CB / 4)
-        reinterpret_cast<float4 *>(vs)[idx] = c0 / 4 + idx % (CB / 4) < dv4 ? raw_to_f4<T>(rv[e]) : make_float4(0.f, 0.f, 0.f, 0.f);
-    }
-    __syncthreads();
-    if (t0 + CR_TT < p.S) fetch(t0 + CR_TT);  // in flight while this chunk is computed
-    if (nt == CR_TT) {
-#pragma unroll 4
-      for (int tt = 0; tt < CR_TT; tt++) token(tt);
-    } else {
-      for (int tt = 0; tt < nt; tt++) token(tt);
-    }
+    asm volatile("cp.async.wait_group 0;" ::: "memory");
+    __syncthreads();  // this chunk has landed; the other buffer and the partial outputs of the chunk before are free
+    if (t0 + CR_TT < p.S) fetch(t0 + CR_TT, stage ^ 1);
+    const float *as = reinterpret_cast<const float *>(raw + stage * C::STAGE);
+    const T *qs = reinterpret_cast<const T *>(as + CR_TT * DK), *ks = qs + CR_TT * DK, *vs = ks + CR_TT * DK;
+    for (int t4 = 0; t4 < nt; t4 += 4) four(as, qs, ks, vs, t4);
     __syncthreads();
     for (int idx = threadIdx.x; idx < nt * CB; idx += 256) {
       const int tt = idx / CB, j = idx % CB;
       float o = 0.f;
 #pragma unroll
       for (int w = 0; w < RW; w++) o += part[(w * CR_TT + tt) * CB + j];
-      if (c0 + j < p.dv) p.o[((m0 + tt) * p.heads + h) * p.dv + c0 + j] = o;
+      if (c0 + j < p.dv) p.o[((m0 + tt) * p.heads + h) * p.dv + c0 + j] = o * p.qscale;  // the output is linear in q
     }
   }
   if (live)
@@ -386,18 +379,22 @@ __global__ void __launch_bounds__(256) recurrence_channels_kernel(const Recurren
     for (int r = 0; r < 4; r++) *reinterpret_cast<float4 *>(gs + (size_t)r * p.dv) = make_float4(St[r][0], St[r][1], St[r][2], St[r][3]);
 }
 template <typename T, int RW> static cudaError_t launch_recurrence_channels(cudaStream_t st, const Recurrence &p) {
-  constexpr int CB = 8 / RW * 16;
-  const size_t smem = (size_t)(3 * CR_TT * RW * 32 + CR_TT * CB + RW * CR_TT * CB) * sizeof(float);
-  if (smem > 48 * 1024) {
-    cudaError_t e = cudaFuncSetAttribute(recurrence_channels_kernel<T, RW>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+  typedef ChannelTile<T, RW> C;
+  static_assert(C::SMEM <= 227 * 1024, "the two buffers and the partial outputs fit an SM");
+  static int attr_dev = -1;  // per instantiation: the device the attribute was last set on (the value never changes)
+  int dev = 0;
+  cudaGetDevice(&dev);
+  if (C::SMEM > 48 * 1024 && attr_dev != dev) {
+    cudaError_t e = cudaFuncSetAttribute(recurrence_channels_kernel<T, RW>, cudaFuncAttributeMaxDynamicSharedMemorySize, C::SMEM);
     if (e != cudaSuccess) return e;
+    attr_dev = dev;
   }
-  recurrence_channels_kernel<T, RW><<<dim3(p.heads * ((p.dv + CB - 1) / CB), p.B), 256, smem, st>>>(p);
+  recurrence_channels_kernel<T, RW><<<dim3(p.heads * ((p.dv + C::CB - 1) / C::CB), p.B), 256, C::SMEM, st>>>(p);
   return cudaSuccess;
 }
 int recurrence_channels(cudaStream_t st, int dtype, const Recurrence &p) {
   const uintptr_t in_align = dtype == 2 ? 15 : 7;
-  if (p.dk > 256 || p.dk % 4 || p.dv % 4 || p.ldq % 4 || p.ldk % 4 || p.ldv % 4 || p.group_div != 1 ||
+  if (p.dk > 256 || p.dk % 4 || p.dv % 4 || p.ldq % 4 || p.ldk % 4 || p.ldv % 4 || p.group_div != 1 || p.kscale != 1.f ||
       (((uintptr_t)p.q | (uintptr_t)p.k | (uintptr_t)p.v) & in_align) || (((uintptr_t)p.a_chan | (uintptr_t)p.state) & 15))
     return (int)cudaErrorNotSupported;
   cudaError_t e = cudaSuccess;
