@@ -940,6 +940,10 @@ __global__ void __launch_bounds__(128) moe_router_kernel(const MoePlan p) {
       ch[sI] = z[sI];
       continue;
     }
+    if (p.sigmoid_scores && !corr) {  // the sigmoid keeps the logits' order where its fp32 value saturates
+      ch[sI] = z[sI];
+      continue;
+    }
     if (!p.sigmoid_scores) sc[sI] = sc[sI] / sum;
     ch[sI] = e < E ? sc[sI] + (corr ? DT<T>::to_f(corr[e]) : 0.f) : -INFINITY;
   }

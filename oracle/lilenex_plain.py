@@ -152,9 +152,10 @@ def expert(h, wt, p):
 
 
 def route(z, top):
-    """z [S, E] router logits -> (experts [S, top], weights [S, top]): sigmoid scores, the largest ones, as they are."""
-    s = torch.sigmoid(z)
-    w, idx = torch.topk(s, top, -1)
+    """z [S, E] router logits -> (experts [S, top], weights [S, top]): the largest sigmoid scores (chosen by logit, which orders them
+    where their rounded values are equal), as they are."""
+    idx = torch.topk(z, top, -1).indices
+    w = torch.sigmoid(torch.gather(z, 1, idx))
     if FAULT == "renormalised":
         w = w / w.sum(-1, keepdim=True)
     return idx, w

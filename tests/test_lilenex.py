@@ -606,9 +606,11 @@ def test_strong_decays_and_saturated_routers():
     for i in (0, 1):
         n = sd[f"l{i}.mix.a2.b"].numel()
         sd[f"l{i}.mix.a2.b"] = torch.linspace(-30.0, 30.0, n)
-    sd["l0.mlp.router"] = sd["l0.mlp.router"] * 3.0
+    sd["l0.mlp.router"] = sd["l0.mlp.router"] * 12.0      # several scores round to one: the logits decide
     toks = tokens(50, cfg.vocab_size, seed=16)
     want = plain(cfg, sd, toks)
+    h = torch.randn(400, 44)
+    assert ((torch.sigmoid(P.lin(sd["l0.mlp.router"], h)) == 1.0).sum(-1) > 2).any()
     r = Runner(cfg, sd, "f32")
     try:
         close(r.run("w", toks), want, "f32", "whole")
