@@ -513,7 +513,7 @@ def test_tiled_attention_of_other_head_sizes():
     """16-bit portions whose head sizes are multiples of eight but not 128, unequal for keys and values: the tiled kernel."""
     layers = [attn(heads=2, kv_heads=1, dim=24, vdim=40, size=9, keep=2, scale=0.05, rot=16, base=1000.0, scaling=None, mlp=None),
               attn(heads=4, kv_heads=1, dim=24, vdim=40, size=80, keep=1, scale=0.05, rot=16, base=1000.0, scaling=None, kv_from=0, mlp=dense(64)),
-              gla(heads=2, dim=48, vdim=64, mlp=moe(8, 2, 64, 64)), attn(heads=3, kv_heads=3, dim=96, vdim=96, size=65, keep=70, scale=0.05, rot=96, mlp=None)]
+              gla(heads=2, dim=40, vdim=72, mlp=moe(8, 2, 64, 64)), attn(heads=3, kv_heads=3, dim=96, vdim=96, size=65, keep=70, scale=0.05, rot=96, mlp=None)]
     cfg, sd, toks, want, bar = f16_case(layers, 128, 128, 330, 48, ("window+1", "window-1", "keep+1", "keep-1", "keep none"))
     r = Runner(cfg, sd, "f16")
     try:
